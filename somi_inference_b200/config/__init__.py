@@ -4,6 +4,8 @@ from .dapozen import ARCHITECTURE as DAPOZEN_ARCHITECTURE
 from .dapozen import DapozenConfig
 from .digosun import ARCHITECTURE as DIGOSUN_ARCHITECTURE
 from .digosun import DigosunConfig
+from .dosuvik import ARCHITECTURE as DOSUVIK_ARCHITECTURE
+from .dosuvik import DosuvikConfig
 from .gikarax import ARCHITECTURE as GIKARAX_ARCHITECTURE
 from .gikarax import GikaraxConfig
 from .poselorn import ARCHITECTURE as POSELORN_ARCHITECTURE
@@ -19,9 +21,11 @@ register_architecture(DIGOSUN_ARCHITECTURE, DigosunConfig)
 register_architecture(DAPOZEN_ARCHITECTURE, DapozenConfig)
 register_architecture(POSELORN_ARCHITECTURE, PoselornConfig)
 register_architecture(GIKARAX_ARCHITECTURE, GikaraxConfig)
+register_architecture(DOSUVIK_ARCHITECTURE, DosuvikConfig)
 
 __all__ = ["ConfigError", "Qwen2Config", "QWEN2_ARCHITECTURE", "DigosunConfig",
            "DIGOSUN_ARCHITECTURE", "DapozenConfig", "DAPOZEN_ARCHITECTURE", "PoselornConfig",
-           "POSELORN_ARCHITECTURE", "GikaraxConfig", "GIKARAX_ARCHITECTURE", "LayerSpec", "ModelSpec",
-           "PartSpec", "RunSpec", "config_class_for", "load_config",
-           "register_architecture", "supported_architectures", "unregister_architecture"]
+           "POSELORN_ARCHITECTURE", "GikaraxConfig", "GIKARAX_ARCHITECTURE", "DosuvikConfig",
+           "DOSUVIK_ARCHITECTURE", "LayerSpec", "ModelSpec", "PartSpec", "RunSpec",
+           "config_class_for", "load_config", "register_architecture", "supported_architectures",
+           "unregister_architecture"]

@@ -61,12 +61,17 @@ class RunSpec:
     before the first run) is added to the stream once more right in front of this run.
     `remix`: the name of one of the model's `stream_parts`; right in front of this run the
     stream is replaced by what that part makes of the stream and the embedding's output.
+    `average`: the name of one of the model's `stream_parts`; behind this run the stream is replaced
+    by what that part makes of the results of all runs so far and the embedding's output.  A model
+    in which some run has one needs one for every run: the record of results is kept by the kernel
+    that takes the average.
     """
 
     layer: int
     cache_of: int | None = None
     add_embedding: bool = False
     remix: str | None = None
+    average: str | None = None
 
 
 @dataclass(frozen=True)
@@ -82,7 +87,7 @@ class ModelSpec:
     schedule: tuple[RunSpec, ...]
     final_norm: PartSpec
     head: PartSpec
-    # parts that act on the residual stream between runs (see `RunSpec.remix`), by name
+    # parts that act on the residual stream between runs (see `RunSpec.remix`, `.average`), by name
     stream_parts: Mapping[str, PartSpec] = field(default_factory=dict)
 
     def validate(self) -> None:
@@ -97,6 +102,9 @@ class ModelSpec:
             if run.remix is not None and run.remix not in self.stream_parts:
                 raise ValueError(f"schedule[{i}].remix names {run.remix!r}, which is none of the "
                                  f"model's stream parts {sorted(self.stream_parts)}")
+            if run.average is not None and run.average not in self.stream_parts:
+                raise ValueError(f"schedule[{i}].average names {run.average!r}, which is none of the "
+                                 f"model's stream parts {sorted(self.stream_parts)}")
             if run.add_embedding and i == 0:
                 raise ValueError("schedule[0] cannot add the embedding's output again")
             if run.cache_of is not None:
@@ -106,3 +114,9 @@ class ModelSpec:
                 if self.schedule[run.cache_of].cache_of is not None:
                     raise ValueError(f"schedule[{i}].cache_of={run.cache_of} names "
                                      "a run that owns no cache")
+        averaged = [run.average is not None for run in self.schedule]
+        if any(averaged) and not all(averaged):
+            raise ValueError("a schedule averages the stream behind every run or behind none")
+        if any(averaged) and any(run.add_embedding or run.remix for run in self.schedule):
+            raise ValueError("a schedule that averages over depth neither re-mixes the stream nor "
+                             "adds the embedding's output again")

@@ -4,12 +4,15 @@
 // (q'_h = W_uk,h^T q_h, so that q_h . k_h = q'_h . c) and applies the value expansion to the
 // result (W_uv,h sum_j p_j c_j), which is why only the latent c is cached.
 //
+// A cache row may end with a part that only the scores read (a rotated key part shared by the
+// heads): rows are R wide, of which the first V are the values.
+//
 //   s_ij = scale * q'_i . c_j          for max(0, i - window + 1) <= j <= i   (window 0: all j <= i)
 //   p_ij = exp(s_ij - m_i) / (sum_j exp(s_ij - m_i) + exp(sink_h - m_i)),  m_i = max(sink_h, max_j s_ij)
-//   o_i  = sum_j p_ij c_j
+//   o_i  = sum_j p_ij c_j[0..V)
 // The sink adds to the denominator only: a key whose score is sink_h and whose value is zero.
 //
-// This file holds the kernel on the CUDA cores for any dtype and any latent width up to 512 (the
+// This file holds the kernel on the CUDA cores for any dtype, rows of up to 1024 and values of up to 512 (the
 // float32 path's kernel, and the bfloat16 path's for widths the tensor-core kernel of
 // attention_latent_mma.cu refuses).
 // Key tiles are aligned to multiples of kBN from position 0 and the softmax is online in
@@ -25,8 +28,9 @@ namespace somi {
 constexpr int kLBM = 16;
 constexpr int kLBN = 32;
 constexpr int kLThreads = 128;
-constexpr int kLMaxR = 512;
-constexpr int kLAcc = kLBM * kLMaxR / kLThreads;     // 64
+constexpr int kLMaxR = 1024;
+constexpr int kLMaxV = 512;
+constexpr int kLAcc = kLBM * kLMaxV / kLThreads;     // 64
 
 template <typename T>
 __global__ void __launch_bounds__(kLThreads)
@@ -35,7 +39,7 @@ latent_attention_generic_kernel(const T* __restrict__ q, long long q_tok_stride,
                                 const int* __restrict__ block_table, int bt_stride,
                                 const int* __restrict__ cu_q, const int* __restrict__ ctx_len,
                                 const int* __restrict__ tiles, int n_tiles, int n_prefill_req,
-                                int n_prefill_tok, int R, int page_size, float scale, int window,
+                                int n_prefill_tok, int R, int V, int page_size, float scale, int window,
                                 const float* __restrict__ sinks, T* __restrict__ out,
                                 long long o_tok_stride, long long o_head_stride) {
     extern __shared__ float smem[];
@@ -132,8 +136,8 @@ latent_attention_generic_kernel(const T* __restrict__ q, long long q_tok_stride,
 #pragma unroll
         for (int i = 0; i < kLAcc; ++i) {
             const int idx = tid + i * kLThreads;
-            if (idx < kLBM * R) {
-                const int m = idx / R, d = idx - m * R;
+            if (idx < kLBM * V) {
+                const int m = idx / V, d = idx - m * V;
                 float o = acc[i] * a_s[m];
                 const float* p = Ss + m * (kLBN + 1);
 #pragma unroll 4
@@ -146,8 +150,8 @@ latent_attention_generic_kernel(const T* __restrict__ q, long long q_tok_stride,
 #pragma unroll
     for (int i = 0; i < kLAcc; ++i) {
         const int idx = tid + i * kLThreads;
-        if (idx < kLBM * R) {
-            const int m = idx / R, d = idx - m * R;
+        if (idx < kLBM * V) {
+            const int m = idx / V, d = idx - m * V;
             if (m < rows)
                 out[static_cast<size_t>(row0 + m) * o_tok_stride +
                     static_cast<size_t>(head) * o_head_stride + d] = from_float<T>(acc[i] / l_s[m]);
@@ -162,15 +166,15 @@ using namespace somi;
 SOMI_API int somi_latent_attention_generic_q_tile() { return kLBM; }
 
 // q, out: element (token t, head h, d) at t * tok_stride + h * head_stride + d.
-// cache: [pages, page_size, R].  sinks: float32 [heads] or null.
+// q rows: R wide, out rows: V <= R wide; cache: [pages, page_size, R].  sinks: float32 [heads] or null.
 SOMI_API int somi_latent_attention_generic(
     const void* q, int dtype, long long q_tok_stride, long long q_head_stride, const void* cache,
     const int* block_table, int bt_stride, const int* cu_q, const int* ctx_len, const int* tiles,
     int n_tiles, int n_prefill_req, int n_prefill_tok, int n_decode, int heads, int R,
-    int page_size, float scale, int window, const float* sinks, void* out, long long o_tok_stride,
+    int V, int page_size, float scale, int window, const float* sinks, void* out, long long o_tok_stride,
     long long o_head_stride, cudaStream_t stream) {
     if (n_tiles + n_decode <= 0) return 0;
-    if (R <= 0 || R > kLMaxR || heads <= 0 || heads > 65535 || page_size <= 0)
+    if (R <= 0 || R > kLMaxR || V <= 0 || V > kLMaxV || V > R || heads <= 0 || heads > 65535 || page_size <= 0)
         return SOMI_ERR_UNSUPPORTED;
     const size_t smem = sizeof(float) * (static_cast<size_t>(kLBM) * R + kLBN * (R + 1) +
                                          kLBM * (kLBN + 1) + 3 * kLBM);
@@ -183,7 +187,7 @@ SOMI_API int somi_latent_attention_generic(
         launch_pdl(latent_attention_generic_kernel<T>, dim3(grid), dim3(kLThreads), smem,       \
             stream, static_cast<const T*>(q), q_tok_stride, q_head_stride,                      \
             static_cast<const T*>(cache), block_table, bt_stride, cu_q, ctx_len, tiles,         \
-            n_tiles, n_prefill_req, n_prefill_tok, R, page_size, scale, window, sinks,          \
+            n_tiles, n_prefill_req, n_prefill_tok, R, V, page_size, scale, window, sinks,          \
             static_cast<T*>(out), o_tok_stride, o_head_stride);                                 \
     } while (0)
     if (dtype == SOMI_F32) SOMI_LAUNCH_LATT(float);

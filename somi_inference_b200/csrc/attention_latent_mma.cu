@@ -12,9 +12,10 @@
 //     chunks of `chunk` positions, one CTA (blockIdx.z) each, whose partial sums (float32, with
 //     their maximum and denominator) a merge kernel adds up; with one chunk the CTA writes the
 //     result itself.
-// RT is the latent width rounded up to 64/128/256/512 (columns beyond the width are zeros in
-// shared memory).  Up to RT = 256 a warp owns 16 rows and all columns of O (four warps); at
-// RT = 512 two warps share a row tile (eight warps: registers hold 16 x 256 accumulators at
+// A cache row is R wide, of which the first V columns are the values (R > V: a key part that only
+// the scores read lies behind them).  RT is R rounded up to 64/128/256/512/576 (columns beyond the
+// width are zeros in shared memory), VT the columns of O that are computed (RT, or 512 at 576).  Up to RT = 256 a warp owns 16 rows and all columns of O (four warps); at
+// RT = 512 and 576 two warps share a row tile (eight warps: registers hold 16 x 256 accumulators at
 // most): each computes the scores of half of a tile's keys, they exchange row maxima, row sums
 // and P (in the MMA's register layout) through shared memory at two barriers of their own, and
 // each accumulates half of the output columns.  Softmax: online, float32,
@@ -55,16 +56,20 @@ __device__ __forceinline__ void load_latent_tile(unsigned char* dst,
 __device__ __forceinline__ void pair_barrier(int mt) {
     asm volatile("bar.sync %0, 64;\n" ::"r"(mt + 1) : "memory");
 }
-constexpr int kLtExchangeBytes = 4096 + 4 * 2 * 2 * 4 * 32 * 4;     // maxima, sums, P (12 KB)
+// what they exchange: maxima, sums, P (12 KB); rows wider than 512 leave no room for the sums, which
+// each warp then takes from its partner's P
+__host__ __device__ constexpr int latent_exchange_bytes(int RT) {
+    return (RT > 512 ? 2048 : 4096) + 4 * 2 * 2 * 4 * 32 * 4;
+}
 
-template <int RT, int CSPLIT>
+template <int RT, int VT, int CSPLIT>
 __global__ void __launch_bounds__(128 * CSPLIT)
 latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_tok_stride,
                             long long q_head_stride, const __nv_bfloat16* __restrict__ cache,
                             const int* __restrict__ block_table, int bt_stride,
                             const int* __restrict__ cu_q, const int* __restrict__ ctx_len,
                             const int* __restrict__ tiles, int req_base, int row_base, int tokb,
-                            int H, int R, int page_size, float scale_log2e, int window,
+                            int H, int R, int V, int page_size, float scale_log2e, int window,
                             const float* __restrict__ sinks, __nv_bfloat16* __restrict__ out,
                             long long o_tok_stride, long long o_head_stride, int chunk,
                             float* __restrict__ part_o, float* __restrict__ part_ml,
@@ -72,7 +77,8 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_tok
     constexpr int CPR = RT / 8;
     constexpr int TILE = kLtBN * RT * 2;
     constexpr int THREADS = 128 * CSPLIT;
-    constexpr int OC = RT / 8 / CSPLIT;                 // 8-column output tiles per warp
+    constexpr int OC = VT / 8 / CSPLIT;                 // 8-column output tiles per warp
+    constexpr bool kOwnSums = RT > 512;
     extern __shared__ __align__(128) unsigned char smem_raw[];
     unsigned char* Qs = smem_raw;                        // [64][RT]
     unsigned char* Cs = Qs + kLtRows * RT * 2;           // 2 x [64][RT]
@@ -232,14 +238,31 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_tok
                 // P of this warp's keys, in the MMA's own register layout (both warps of a row
                 // tile hold the same rows in the same lanes), and its row sums
                 float2* xsum = reinterpret_cast<float2*>(xch + 2048) + (mt * 2) * 32;
-                uint32_t* xp = reinterpret_cast<uint32_t*>(xch + 4096) + (mt * 2) * (NP * 4 * 32);
-                xsum[cs * 32 + lane] = make_float2(r_lo, r_hi);
+                uint32_t* xp = reinterpret_cast<uint32_t*>(xch + (kOwnSums ? 2048 : 4096)) + (mt * 2) * (NP * 4 * 32);
+                if constexpr (!kOwnSums) xsum[cs * 32 + lane] = make_float2(r_lo, r_hi);
 #pragma unroll
                 for (int k = 0; k < NP; ++k)
 #pragma unroll
                     for (int e = 0; e < 4; ++e) xp[cs * (NP * 4 * 32) + (k * 4 + e) * 32 + lane] = own[k][e];
                 pair_barrier(mt);
-                const float2 other = xsum[(cs ^ 1) * 32 + lane];
+                float2 other = make_float2(0.f, 0.f);
+                if constexpr (!kOwnSums) other = xsum[(cs ^ 1) * 32 + lane];
+                if constexpr (kOwnSums) {
+                    // the partner's row sums, added in the partner's order
+#pragma unroll
+                    for (int k = 0; k < NP; ++k)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            const uint32_t w = xp[(cs ^ 1) * (NP * 4 * 32) + (k * 4 + e) * 32 + lane];
+                            const __nv_bfloat162 p = *reinterpret_cast<const __nv_bfloat162*>(&w);
+                            const float s2 = __low2float(p) + __high2float(p);
+                            if (e & 1) other.y += s2; else other.x += s2;
+                        }
+                    other.x += __shfl_xor_sync(0xffffffffu, other.x, 1);
+                    other.x += __shfl_xor_sync(0xffffffffu, other.x, 2);
+                    other.y += __shfl_xor_sync(0xffffffffu, other.y, 1);
+                    other.y += __shfl_xor_sync(0xffffffffu, other.y, 2);
+                }
                 // the same order of addition in both warps: first half's keys, then second half's
                 r_lo = cs == 0 ? r_lo + other.x : other.x + r_lo;
                 r_hi = cs == 0 ? r_hi + other.y : other.y + r_hi;
@@ -280,7 +303,7 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_tok
 #pragma unroll
         for (int nt = 0; nt < OC; ++nt) {
             const int d = (cs * OC + nt) * 8 + (lane & 3) * 2;
-            if (d >= R) continue;
+            if (d >= V) continue;
             if (ok_lo)
                 *reinterpret_cast<uint32_t*>(out + static_cast<size_t>(row0 + row_lo % tokb) * o_tok_stride +
                                              static_cast<size_t>(head_lo) * o_head_stride + d) =
@@ -299,9 +322,9 @@ latent_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, long long q_tok
 #pragma unroll
     for (int nt = 0; nt < OC; ++nt) {
         const int d = (cs * OC + nt) * 8 + (lane & 3) * 2;
-        if (d >= R) continue;
-        if (ok_lo) *reinterpret_cast<float2*>(part_o + p_lo * R + d) = make_float2(o[nt][0], o[nt][1]);
-        if (ok_hi) *reinterpret_cast<float2*>(part_o + p_hi * R + d) = make_float2(o[nt][2], o[nt][3]);
+        if (d >= V) continue;
+        if (ok_lo) *reinterpret_cast<float2*>(part_o + p_lo * V + d) = make_float2(o[nt][0], o[nt][1]);
+        if (ok_hi) *reinterpret_cast<float2*>(part_o + p_hi * V + d) = make_float2(o[nt][2], o[nt][3]);
     }
     if (cs == 0 && (lane & 3) == 0) {
         if (ok_lo) *reinterpret_cast<float2*>(part_ml + 2 * p_lo) = make_float2(m_lo, l_lo);
@@ -340,22 +363,24 @@ __global__ void latent_merge_kernel(const float* __restrict__ part_o, const floa
     }
 }
 
-template <int RT, int CSPLIT>
+template <int RT, int VT, int CSPLIT>
 int launch_latent_mma(dim3 grid, cudaStream_t stream, const void* q, long long qts, long long qhs,
                       const void* cache, const int* block_table, int bt_stride, const int* cu_q,
                       const int* ctx_len, const int* tiles, int req_base, int row_base, int tokb,
-                      int H, int R, int page_size, float scale, int window, const float* sinks,
+                      int H, int R, int V, int page_size, float scale, int window, const float* sinks,
                       void* out, long long ots, long long ohs, int chunk, float* part_o,
                       float* part_ml, int max_splits) {
     const size_t smem = static_cast<size_t>(kLtRows + 2 * kLtBN) * RT * 2 +
-                        (CSPLIT == 2 ? kLtExchangeBytes : 0);
+                        (CSPLIT == 2 ? latent_exchange_bytes(RT) : 0);
+    static_assert((kLtRows + 2 * kLtBN) * RT * 2 + (CSPLIT == 2 ? latent_exchange_bytes(RT) : 0) <= 227 * 1024,
+                  "tiles and exchange must fit into shared memory");
     if (smem > 48 * 1024)
-        cudaFuncSetAttribute(latent_attention_mma_kernel<RT, CSPLIT>,
+        cudaFuncSetAttribute(latent_attention_mma_kernel<RT, VT, CSPLIT>,
                              cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return launch_pdl(latent_attention_mma_kernel<RT, CSPLIT>, grid, dim3(128 * CSPLIT), smem, stream,
+    return launch_pdl(latent_attention_mma_kernel<RT, VT, CSPLIT>, grid, dim3(128 * CSPLIT), smem, stream,
                       static_cast<const __nv_bfloat16*>(q), qts, qhs,
                       static_cast<const __nv_bfloat16*>(cache), block_table, bt_stride, cu_q, ctx_len,
-                      tiles, req_base, row_base, tokb, H, R, page_size,
+                      tiles, req_base, row_base, tokb, H, R, V, page_size,
                       scale * 1.4426950408889634f, window, sinks, static_cast<__nv_bfloat16*>(out),
                       ots, ohs, chunk, part_o, part_ml, max_splits);
 }
@@ -365,14 +390,15 @@ int launch_latent_mma(dim3 grid, cudaStream_t stream, const void* q, long long q
 using namespace somi;
 
 SOMI_API int somi_latent_attention_mma_q_tile() { return 16; }
-SOMI_API int somi_latent_attention_mma_supported(int heads, int R) {
-    return heads >= 1 && heads <= 65535 * 4 && R >= 8 && R <= 512 && R % 8 == 0;
+SOMI_API int somi_latent_attention_mma_supported(int heads, int R, int V) {
+    return heads >= 1 && heads <= 65535 * 4 && R >= 8 && R <= 576 && R % 8 == 0 && V >= 8 && V <= R &&
+           V <= 512 && V % 8 == 0;
 }
 
 // bfloat16.  `tiles`: int32 [n_tiles, 3] = (request, first row, rows <= 16) over the multi-token
 // requests; the n_decode single-token requests follow them (request n_prefill_req + i, row
 // n_prefill_tok + i).  `max_kv_len`: the longest request's keys after this step.  `scratch`:
-// float32, at least n_decode * heads * splits * (R + 2) elements where splits =
+// float32, at least n_decode * heads * splits * (V + 2) elements where splits =
 // somi_latent_attention_mma_splits(max_kv_len, window, n_decode, heads) > 1.
 // Keys per chunk of a single-token request: a multiple of the key tile, as small as keeps the
 // step's CTAs (requests x head groups x chunks) within two per SM.  A short chunk means a short
@@ -395,10 +421,10 @@ SOMI_API int somi_latent_attention_mma(
     const void* q, long long q_tok_stride, long long q_head_stride, const void* cache,
     const int* block_table, int bt_stride, const int* cu_q, const int* ctx_len, const int* tiles,
     int n_tiles, int n_prefill_req, int n_prefill_tok, int n_decode, int max_kv_len, int heads,
-    int R, int page_size, float scale, int window, const float* sinks, void* out,
+    int R, int V, int page_size, float scale, int window, const float* sinks, void* out,
     long long o_tok_stride, long long o_head_stride, float* scratch, cudaStream_t stream) {
     if (n_tiles + n_decode <= 0) return 0;
-    if (!somi_latent_attention_mma_supported(heads, R) || page_size <= 0 ||
+    if (!somi_latent_attention_mma_supported(heads, R, V) || page_size <= 0 ||
         (q_tok_stride | q_head_stride | o_tok_stride | o_head_stride) % 8 ||
         (reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) % 16)
         return SOMI_ERR_UNSUPPORTED;
@@ -406,32 +432,33 @@ SOMI_API int somi_latent_attention_mma(
     const int chunk = latent_chunk(max_kv_len, window, n_decode, heads);
     if (splits > 65535) return SOMI_ERR_UNSUPPORTED;
     float* part_o = scratch;
-    float* part_ml = scratch ? scratch + static_cast<size_t>(n_decode) * heads * splits * R : nullptr;
+    float* part_ml = scratch ? scratch + static_cast<size_t>(n_decode) * heads * splits * V : nullptr;
     if (splits > 1 && !scratch) return SOMI_ERR_UNSUPPORTED;
     int rc = 0;
-#define SOMI_LATT_MMA(RT, CS)                                                                   \
+#define SOMI_LATT_MMA(RT, VT, CS)                                                                   \
     do {                                                                                        \
         if (n_tiles > 0)                                                                        \
-            rc = launch_latent_mma<RT, CS>(dim3(n_tiles, (heads + 3) / 4), stream, q,           \
+            rc = launch_latent_mma<RT, VT, CS>(dim3(n_tiles, (heads + 3) / 4), stream, q,           \
                 q_tok_stride, q_head_stride, cache, block_table, bt_stride, cu_q, ctx_len,      \
-                tiles, 0, 0, 16, heads, R, page_size, scale, window, sinks, out, o_tok_stride,  \
+                tiles, 0, 0, 16, heads, R, V, page_size, scale, window, sinks, out, o_tok_stride,  \
                 o_head_stride, 0, nullptr, nullptr, 1);                                         \
         if (rc == 0 && n_decode > 0)                                                            \
-            rc = launch_latent_mma<RT, CS>(dim3(n_decode, (heads + 63) / 64, splits), stream,   \
+            rc = launch_latent_mma<RT, VT, CS>(dim3(n_decode, (heads + 63) / 64, splits), stream,   \
                 q, q_tok_stride, q_head_stride, cache, block_table, bt_stride, cu_q, ctx_len,   \
-                nullptr, n_prefill_req, n_prefill_tok, 1, heads, R, page_size, scale, window,   \
+                nullptr, n_prefill_req, n_prefill_tok, 1, heads, R, V, page_size, scale, window,   \
                 sinks, out, o_tok_stride, o_head_stride, splits > 1 ? chunk : 0, part_o, part_ml,\
                 splits);                                                                        \
     } while (0)
-    if (R <= 64) SOMI_LATT_MMA(64, 1);
-    else if (R <= 128) SOMI_LATT_MMA(128, 1);
-    else if (R <= 256) SOMI_LATT_MMA(256, 1);
-    else SOMI_LATT_MMA(512, 2);
+    if (R <= 64) SOMI_LATT_MMA(64, 64, 1);
+    else if (R <= 128) SOMI_LATT_MMA(128, 128, 1);
+    else if (R <= 256) SOMI_LATT_MMA(256, 256, 1);
+    else if (R <= 512) SOMI_LATT_MMA(512, 512, 2);
+    else SOMI_LATT_MMA(576, 512, 2);
 #undef SOMI_LATT_MMA
     if (rc != 0) return rc;
     if (n_decode > 0 && splits > 1)
-        launch_pdl(latent_merge_kernel, dim3(n_decode, heads), dim3(min(256, ((R + 31) / 32) * 32)), 0,
-                   stream, part_o, part_ml, splits, splits, heads, R, sinks, n_prefill_tok,
+        launch_pdl(latent_merge_kernel, dim3(n_decode, heads), dim3(min(256, ((V + 31) / 32) * 32)), 0,
+                   stream, part_o, part_ml, splits, splits, heads, V, sinks, n_prefill_tok,
                    static_cast<__nv_bfloat16*>(out), o_tok_stride, o_head_stride);
     return launch_status();
 }

@@ -30,6 +30,9 @@ constexpr int kGemmWBytes = kGemmBN * kGemmBK * 2;      // 16 KiB
 
 enum GemmMode { kGemmBf16 = 0, kGemmF32 = 1, kGemmPartialF32 = 2, kGemmSwiGLU = 3, kGemmXieluSide = 4 };
 
+// the gated activation of kGemmSwiGLU (limit infinite, alpha 1, shift 0: silu(gate) * up)
+struct GluForm { float limit, alpha, shift; };
+
 __device__ int g_gemm_error = 0;
 
 __device__ __forceinline__ uint64_t umma_smem_desc(uint32_t smem_addr) {
@@ -78,7 +81,7 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap w_map,
                    const __grid_constant__ CUtensorMap x_map, int M, int N, int K,
                    int kb_per_split, int mode, const void* __restrict__ bias, int bias_dtype,
                    void* __restrict__ out, long long out_split_stride, void* __restrict__ out2,
-                   int n_act, const float* __restrict__ act) {
+                   int n_act, const float* __restrict__ act, GluForm glu) {
     // The two MMA threads take the K blocks in turn.  With an even number of stages each stage
     // belongs to one of them for good, and that thread sees every phase of the stage's barrier in
     // order.  With an odd number a stage would alternate between the threads: a thread could meet
@@ -263,7 +266,8 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap w_map,
                         }
                     }
                 }
-            } else {   // kGemmSwiGLU: even rows of W are gate rows, odd rows the matching up rows
+            } else {   // kGemmSwiGLU: even rows of W are gate rows, odd rows the matching up rows;
+                // g * sigmoid(alpha g) * (u + shift), g = min(gate, limit), u = clamp(up, -limit, limit)
                 __nv_bfloat16* y = static_cast<__nv_bfloat16*>(out);
                 const int half_n = N >> 1;
 #pragma unroll
@@ -271,9 +275,10 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap w_map,
                     if (m >= M) break;                      // uniform: M is a kernel argument
                     const float other = __shfl_xor_sync(0xffffffffu, acc[m], 1);
                     if ((lane & 1) == 0 && n < N) {
-                        const float g = acc[m];
+                        const float g = fminf(acc[m], glu.limit);
+                        const float u = fminf(fmaxf(other, -glu.limit), glu.limit) + glu.shift;
                         y[static_cast<size_t>(m) * half_n + (n >> 1)] =
-                            __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-g)) * other);
+                            __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-glu.alpha * g)) * u);
                     }
                 }
             }
@@ -292,8 +297,8 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap w_map,
 template <int TOK, int STAGES>
 int launch_skinny(const CUtensorMap* w_map, const CUtensorMap* x_map, int M, int N, int K,
                   int splits, int mode, const void* bias, int bias_dtype, void* out,
-                  long long out_split_stride, cudaStream_t stream, void* out2 = nullptr,
-                  int n_act = 0, const float* act = nullptr) {
+                  long long out_split_stride, cudaStream_t stream, void* out2,
+                  int n_act, const float* act, GluForm glu) {
     constexpr int StageBytes = kGemmWBytes + TOK * kGemmBK * 2;
     const size_t smem = static_cast<size_t>(STAGES) * StageBytes + 1024;
     cudaFuncSetAttribute(skinny_gemm_kernel<TOK, STAGES>,
@@ -303,7 +308,7 @@ int launch_skinny(const CUtensorMap* w_map, const CUtensorMap* x_map, int M, int
     dim3 grid((N + kGemmBN - 1) / kGemmBN, (nkb + kbps - 1) / kbps);
     launch_pdl(skinny_gemm_kernel<TOK, STAGES>, dim3(grid), dim3(kGemmThreads), smem, stream, 
         *w_map, *x_map, M, N, K, kbps, mode, bias, bias_dtype, out, out_split_stride, out2, n_act,
-        act);
+        act, glu);
     return launch_status();
 }
 
@@ -340,26 +345,27 @@ SOMI_API int somi_gemm_error() {
 
 SOMI_API int somi_skinny_gemm_act(const void* w_map, const void* x_map, int x_box_rows, int M, int N,
                                   int K, int splits, int mode, const void* bias, int bias_dtype,
-                                  void* out, void* out2, int n_act, const float* act,
-                                  int deep_ring, cudaStream_t stream);
+                                  void* out, void* out2, int n_act, const float* act, float limit,
+                                  float alpha, float shift, int deep_ring, cudaStream_t stream);
 
 // mode: 0 bf16 [M, N]; 1 float32 [M, N]; 2 float32 partial sums [splits, M, N] (bias in split 0);
-// 3 SwiGLU over interleaved gate/up rows, bf16 [M, N / 2].  `x_box_rows` is the box height the
+// 3 the gated activation (GluForm) over interleaved gate/up rows, bf16 [M, N / 2].  `x_box_rows` is the box height the
 // x tensor map was made with (16, 32 or 64) and must be >= M.
 SOMI_API int somi_skinny_gemm(const void* w_map, const void* x_map, int x_box_rows, int M, int N,
                               int K, int splits, int mode, const void* bias, int bias_dtype,
-                              void* out, int deep_ring, cudaStream_t stream) {
+                              void* out, float limit, float alpha, float shift, int deep_ring,
+                              cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     return somi_skinny_gemm_act(w_map, x_map, x_box_rows, M, N, K, splits, mode, bias, bias_dtype, out,
-                                nullptr, 0, nullptr, deep_ring, stream);
+                                nullptr, 0, nullptr, limit, alpha, shift, deep_ring, stream);
 }
 
 // The same with mode 4: xIELU (its two numbers in `act`, float32) of the first `n_act` features
 // to `out` (bf16 [M, n_act]), the other features, bias added, to `out2` (bf16 [M, N - n_act]).
 SOMI_API int somi_skinny_gemm_act(const void* w_map, const void* x_map, int x_box_rows, int M, int N,
                                   int K, int splits, int mode, const void* bias, int bias_dtype,
-                                  void* out, void* out2, int n_act, const float* act,
-                                  int deep_ring, cudaStream_t stream) {
+                                  void* out, void* out2, int n_act, const float* act, float limit,
+                                  float alpha, float shift, int deep_ring, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (M > x_box_rows || K % 8 != 0 || K <= 0 || mode < 0 || mode > 4) return SOMI_ERR_UNSUPPORTED;
     if (mode == kGemmSwiGLU && (N & 1)) return SOMI_ERR_UNSUPPORTED;
@@ -374,7 +380,7 @@ SOMI_API int somi_skinny_gemm_act(const void* w_map, const void* x_map, int x_bo
     // and epilogue overlap the other's main loop.
 #define SOMI_SKINNY(TOK, ST) \
     return launch_skinny<TOK, ST>(wm, xm, M, N, K, splits, mode, bias, bias_dtype, out, stride, stream, \
-                                  out2, n_act, act)
+                                  out2, n_act, act, GluForm{limit, alpha, shift})
     switch (x_box_rows) {
         case 16: if (deep_ring) SOMI_SKINNY(16, 8); else SOMI_SKINNY(16, 6);
         case 32: if (deep_ring) SOMI_SKINNY(32, 8); else SOMI_SKINNY(32, 4);

@@ -2,9 +2,10 @@
 // its token id in a table of the model (ids given), or its own row of a table that a router filled
 // for this step (ids null).
 //
-//   router:   softmax over the router's logits, a correction added for the choice only, the best
-//             `keep` of `count` groups of neighbouring experts by their best member, the `top` best
-//             members of those; the weights are the softmax values of the chosen.
+//   router:   softmax (or sigmoids) of the router's logits, a correction added for the choice only,
+//             the best `keep` of `count` groups of neighbouring experts by their best member (or the
+//             sum of their two best), the `top` best members of those; the weights are the scores of
+//             the chosen, without the correction.
 //   route:    for every (token, k) pair ("entry" t * top + k) the expert table[row, k]; entries are
 //             grouped by expert (a counting sort in one CTA) and the groups are cut into row tiles.
 //             Experts numbered E and above have no matrices ("identity experts": their output is
@@ -396,10 +397,13 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restri
 // choices among those are written to chosen[t, 0..top) in falling order, their s to weight[t, ..].
 // Equal values go to the lower index.  With `over_chosen` the choice is made on the logits
 // themselves (no correction, no groups) and the weights are the softmax over the chosen logits only.
+// `sigmoid`: s = sigmoid(logits) instead of the softmax; `group_best` 2: a group's score is the sum of
+// its two largest choices (of its only one where it has one member).
 __global__ void moe_router_select_kernel(const float* __restrict__ logits, long long l_stride,
                                          const float* __restrict__ correction, int n, int count,
                                          int keep, int top, int* __restrict__ chosen,
-                                         float* __restrict__ weight, int T, int over_chosen) {
+                                         float* __restrict__ weight, int T, int over_chosen,
+                                         int sigmoid, int group_best) {
     extern __shared__ float rs[];            // per warp: s [n], choice [n], group score [count]
     pdl_launch_dependents();
     pdl_wait();
@@ -416,11 +420,11 @@ __global__ void moe_router_select_kernel(const float* __restrict__ logits, long 
     m = warp_max(m);
     float sum = 0.f;
     for (int i = lane; i < n; i += 32) {
-        const float e = expf(z[i] - m);
+        const float e = sigmoid ? 1.0f / (1.0f + expf(-z[i])) : expf(z[i] - m);
         sv[i] = e;
         sum += e;
     }
-    sum = warp_sum(sum);
+    sum = sigmoid ? 1.0f : warp_sum(sum);
     for (int i = lane; i < n; i += 32) {
         const float p = sv[i] / sum;
         sv[i] = p;
@@ -430,9 +434,13 @@ __global__ void moe_router_select_kernel(const float* __restrict__ logits, long 
     if (count > 1 && keep < count) {
         const int size = n / count;
         for (int g = lane; g < count; g += 32) {
-            float best = -INFINITY;
-            for (int i = 0; i < size; ++i) best = fmaxf(best, cv[g * size + i]);
-            gv[g] = best;
+            float best = -INFINITY, second = -INFINITY;
+            for (int i = 0; i < size; ++i) {
+                const float v = cv[g * size + i];
+                second = fmaxf(second, fminf(best, v));
+                best = fmaxf(best, v);
+            }
+            gv[g] = group_best == 2 && size > 1 ? best + second : best;
         }
         __syncwarp();
         // the (count - keep) worst groups leave: the best `keep` stay, marked by +infinity
@@ -695,17 +703,20 @@ SOMI_API int somi_moe_combine(const void* y, int y_dtype, const int* place, cons
 // logits: float32 [T, l_stride] (n columns read); chosen int32 [T, top], weight float32 [T, top].
 SOMI_API int somi_moe_router_select(const float* logits, long long l_stride, const float* correction,
                                     int T, int n, int count, int keep, int top, int* chosen,
-                                    float* weight, int over_chosen, cudaStream_t stream) {
+                                    float* weight, int over_chosen, int sigmoid, int group_best,
+                                    cudaStream_t stream) {
     if (T <= 0) return 0;
     if (n <= 0 || n > 4096 || top <= 0 || top > n || (count > 1 && (n % count || keep <= 0 || keep > count)))
         return SOMI_ERR_UNSUPPORTED;
     if (count > 1 && keep < count && top > keep * (n / count)) return SOMI_ERR_UNSUPPORTED;
+    if ((sigmoid && over_chosen) || group_best < 1 || group_best > 2) return SOMI_ERR_UNSUPPORTED;
     const int warps = 4;
     const size_t smem = sizeof(float) * warps * (2 * n + (count > 1 ? count : 1));
     if (smem > 48 * 1024)
         cudaFuncSetAttribute(moe_router_select_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_pdl(moe_router_select_kernel, dim3((T + warps - 1) / warps), dim3(32 * warps), smem, stream,
-               logits, l_stride, correction, n, count, keep, top, chosen, weight, T, over_chosen);
+               logits, l_stride, correction, n, count, keep, top, chosen, weight, T, over_chosen, sigmoid,
+               group_best);
     return launch_status();
 }
 

@@ -12,6 +12,7 @@
 // Norms, angles, gates, decays, step sizes and the state are float32; inputs and outputs are float32
 // or bfloat16.
 #include "common.cuh"
+#include "rotation.cuh"
 #include "vec4.cuh"
 
 namespace somi {
@@ -216,8 +217,9 @@ __global__ void headnorm_rotary_store_kernel(T* __restrict__ qkv, long long stri
 //     S <- S + k u^T;   y[t, h, :] = S^T q.
 // q and k of head h are head h / (heads / qk_heads) of their tensors.  With `act_silu` q and k
 // (bit 0) and v (bit 1) pass SiLU as they are read; with `unit` q and k are divided by
-// sqrt(sum of squares + unit_eps); q is multiplied by q_scale either way.  v and beta are read by their
-// own dtype code; with `decay_ready` a holds the decays g themselves.
+// sqrt(sum of squares + unit_eps); q is multiplied by q_scale either way.  With `rot` > 0 entry
+// i < rot / 2 of q and k is paired with entry i + rot / 2 and the pair turns by position * rot_freq[i]
+// before anything else.  v and beta are read by their own dtype code; with `decay_ready` a holds the decays g themselves.
 // A CTA owns kRecCols columns of S for one (request, head) and walks through the request's rows
 // of this step, B rows at a time (16, or 4 when no request has more rows than that).  Four warps
 // hold the state, four columns each, every lane a few rows of all four (RecShape below); the sums
@@ -338,6 +340,17 @@ __device__ __forceinline__ void rec_gather4(float mine, int lane, float (&u)[4])
     u[0] = hi ? x0 : p0; u[1] = hi ? x1 : p1; u[2] = hi ? p0 : x0; u[3] = hi ? p1 : x1;
 }
 
+// Entry i of a head x [.., dk] turned at `pos` (i < rot; its partner lies rot / 2 away)
+template <typename T>
+__device__ __forceinline__ float rec_turned(const T* x, int i, int rot, double pos, const double* freq) {
+    const int half = rot >> 1;
+    const float own = to_float(x[i]);
+    if (i >= rot) return own;
+    const float2 cs = turn_by(pos, freq[i < half ? i : i - half]);
+    return i < half ? fmaf(own, cs.x, -(to_float(x[i + half]) * cs.y))
+                    : fmaf(own, cs.x, to_float(x[i - half]) * cs.y);
+}
+
 template <typename T, int R, bool DELTA, int B>
 __global__ void __launch_bounds__(kRecThreads, R > 16 ? 1 : (B == kRecBlockShort ? 4 : 2))
 matrix_state_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const void* __restrict__ v,
@@ -348,7 +361,8 @@ matrix_state_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const
                          const float* __restrict__ dt_bias, const float* __restrict__ a_log,
                          const float* __restrict__ decay, float* __restrict__ state,
                          const int* __restrict__ cu_q, const int* __restrict__ state_slot,
-                         float* __restrict__ y, int heads, int qk_heads, int dk, int dv) {
+                         float* __restrict__ y, int heads, int qk_heads, int dk, int dv,
+                         const int* __restrict__ positions, const double* __restrict__ rot_freq, int rot) {
     constexpr int DP = R * kRecLanes;                    // padded key width
     constexpr int PL = (DP + 31) / 32;                   // key channels a staging lane holds
     constexpr int V = RecShape<R>::V, RL = RecShape<R>::RL;
@@ -407,8 +421,17 @@ matrix_state_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const
             for (int j = 0; j < PL; ++j) {
                 const int i = lane + 32 * j;
                 const bool in = tok < n_tok && i < dk;
-                qv[m][j] = in ? to_float(q[t * q_stride + static_cast<size_t>(qkh) * dk + i]) : 0.f;
-                kv[m][j] = in ? to_float(k[t * k_stride + static_cast<size_t>(qkh) * dk + i]) : 0.f;
+                const T* qh = q + t * q_stride + static_cast<size_t>(qkh) * dk;
+                const T* kh = k + t * k_stride + static_cast<size_t>(qkh) * dk;
+                // (the launcher has rows of long steps turned by the kernel that makes them ready)
+                if (B == kRecBlockShort && rot > 0) {
+                    const double pos = in ? static_cast<double>(positions[t]) : 0.0;
+                    qv[m][j] = in ? rec_turned(qh, i, rot, pos, rot_freq) : 0.f;
+                    kv[m][j] = in ? rec_turned(kh, i, rot, pos, rot_freq) : 0.f;
+                } else {
+                    qv[m][j] = in ? to_float(qh[i]) : 0.f;
+                    kv[m][j] = in ? to_float(kh[i]) : 0.f;
+                }
                 av[m][j] = (in && channel_decay) ? a[t * a_stride + static_cast<size_t>(h) * dk + i] : 0.f;
             }
         }
@@ -544,7 +567,8 @@ matrix_state_prepare_kernel(const T* __restrict__ q, const T* __restrict__ k, lo
                             const float* __restrict__ a, long long a_stride,
                             const float* __restrict__ dt_bias, const float* __restrict__ a_log,
                             float* __restrict__ qn, float* __restrict__ kn, float* __restrict__ gd,
-                            int rows, int heads, int qk_heads, int dk) {
+                            int rows, int heads, int qk_heads, int dk,
+                            const int* __restrict__ positions, const double* __restrict__ rot_freq, int rot) {
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31;
@@ -571,8 +595,19 @@ matrix_state_prepare_kernel(const T* __restrict__ q, const T* __restrict__ k, lo
     for (int j = 0; j < kRecMaxPL; ++j) {
         const int i = lane + 32 * j;
         const bool in = i < dk;
-        qv[j] = in ? to_float(q[row * q_stride + static_cast<size_t>(qkh) * dk + i]) : 0.f;
-        kv[j] = in ? to_float(k[row * k_stride + static_cast<size_t>(qkh) * dk + i]) : 0.f;
+        const T* qh = q + row * q_stride + static_cast<size_t>(qkh) * dk;
+        const T* kh = k + row * k_stride + static_cast<size_t>(qkh) * dk;
+        if (in && i < rot) {
+            // one sine and cosine for q and k; the arithmetic of rec_turned
+            const int half = rot >> 1, other = i < half ? i + half : i - half;
+            const float2 cs = turn_by(static_cast<double>(positions[t]), rot_freq[i < half ? i : other]);
+            const float sn = i < half ? -cs.y : cs.y;
+            qv[j] = fmaf(to_float(qh[i]), cs.x, to_float(qh[other]) * sn);
+            kv[j] = fmaf(to_float(kh[i]), cs.x, to_float(kh[other]) * sn);
+        } else {
+            qv[j] = in ? to_float(qh[i]) : 0.f;
+            kv[j] = in ? to_float(kh[i]) : 0.f;
+        }
     }
 #pragma unroll
     for (int j = 0; j < kRecMaxPL; ++j) {
@@ -600,7 +635,7 @@ matrix_state_prepare_kernel(const T* __restrict__ q, const T* __restrict__ k, lo
 
 // ------------------------------------------- RMS norm in parts, weight, sigmoid gate
 // The C columns of y[t] in `groups` equal parts of n = C / groups, each divided by its own root
-// mean square; out = that * weight[c % w_len] * sigmoid(gate[t, c]) (gate null: no gate; its rows
+// mean square; out = that * weight[c % w_len] (null: no weight) * sigmoid(gate[t, c]) (gate null: no gate; its rows
 // lie `g_stride` elements apart; gate_act 1: SiLU of the gate instead of its sigmoid).  One CTA per (token, part).
 template <typename TO>
 __global__ void group_rmsnorm_gate_kernel(const float* __restrict__ y, const void* __restrict__ gate,
@@ -620,7 +655,8 @@ __global__ void group_rmsnorm_gate_kernel(const float* __restrict__ y, const voi
     const float r = 1.0f / sqrtf(ss / static_cast<float>(n) + eps);
     TO* o = out + static_cast<size_t>(t) * C + c0;
     for (int i = threadIdx.x; i < n; i += blockDim.x) {
-        float v = yr[i] * r * load_as_float(weight, w_dtype, (c0 + i) % w_len);
+        float v = yr[i] * r;
+        if (weight != nullptr) v *= load_as_float(weight, w_dtype, (c0 + i) % w_len);
         if (gate != nullptr) {
             const float g = load_as_float(gate, g_dtype, static_cast<size_t>(t) * g_stride + c0 + i);
             v *= gate_act == 1 ? silu32(g) : sigmoid32(g);
@@ -663,7 +699,8 @@ group_rmsnorm_gate_warp_kernel(const float* __restrict__ y, const void* __restri
     for (int j = 0; j < kPartWarpMax / 32; ++j) {
         const int i = lane + 32 * j;
         if (i < n) {
-            float z = v[j] * r * load_as_float(weight, w_dtype, (c0 + i) % w_len);
+            float z = v[j] * r;
+            if (weight != nullptr) z *= load_as_float(weight, w_dtype, (c0 + i) % w_len);
             if (gate != nullptr) {
                 const float g = load_as_float(gate, g_dtype, static_cast<size_t>(t) * g_stride + c0 + i);
                 z *= gate_act == 1 ? silu32(g) : sigmoid32(g);
@@ -793,7 +830,8 @@ SOMI_API int somi_matrix_state_scan_max_key() { return 32 * kRecLanes; }
 // q, k: [T, *_stride] with qk_heads heads of dk elements from the pointer on; v: heads heads of dv.
 // delta != 0: beta [T, beta_stride] logits per head, of q's dtype.  a != null: float32 [T, a_stride]
 // decay logits per head and key channel with dt_bias [heads * dk] and a_log [heads]; else
-// decay [heads] (decay_ready: a holds the decays).  dtype: of q and k; vb_dtype: of v and beta.
+// decay [heads] (decay_ready: a holds the decays).  rot > 0 (a step of few rows only): q and k turn by
+// positions [T] * rot_freq [rot / 2].  dtype: of q and k; vb_dtype: of v and beta.
 // state: float32 [slots, heads, dv, dk]; y: float32 [T, heads * dv].  max_rows: the
 // most rows any request has in this step (0: not known); it only chooses how many rows are staged
 // at a time, the sums are the same.
@@ -805,11 +843,16 @@ SOMI_API int somi_matrix_state_scan(const void* q, const void* k, const void* v,
                                     const float* dt_bias, const float* a_log,
                                     const float* decay, float* state, const int* cu_q,
                                     const int* state_slot, float* y, int R, int heads, int qk_heads,
-                                    int dk, int dv, int max_rows, cudaStream_t stream) {
+                                    int dk, int dv, int max_rows, const int* positions,
+                                    const double* rot_freq, int rot, cudaStream_t stream) {
     if (R <= 0) return 0;
     if (dk <= 0 || dk > 32 * kRecLanes || dv <= 0 || heads <= 0 || qk_heads <= 0 || heads % qk_heads ||
         (delta && beta == nullptr) || (a == nullptr && decay == nullptr) ||
         (a != nullptr && (dt_bias == nullptr || a_log == nullptr)))
+        return SOMI_ERR_UNSUPPORTED;
+    // the scan itself turns q and k only where it stages few rows
+    if (rot < 0 || (rot & 1) || rot > dk ||
+        (rot > 0 && (positions == nullptr || rot_freq == nullptr || max_rows <= 0 || max_rows > kRecBlockShort)))
         return SOMI_ERR_UNSUPPORTED;
     dim3 grid(R, heads, (dv + kRecCols - 1) / kRecCols);
     const int rows = (dk + kRecLanes - 1) / kRecLanes;
@@ -821,7 +864,8 @@ SOMI_API int somi_matrix_state_scan(const void* q, const void* k, const void* v,
     launch_pdl(matrix_state_scan_kernel<TT, RR, DD, BB>, grid, dim3(kRecThreads), smem, stream,   \
                static_cast<const TT*>(q), static_cast<const TT*>(k), v, vb_dtype,                 \
                q_stride, k_stride, v_stride, act_silu, unit, unit_eps, q_scale,                 \
-               beta, beta_stride, a, a_stride, decay_ready, dt_bias, a_log, decay, state, cu_q, state_slot, y, heads, qk_heads, dk, dv)
+               beta, beta_stride, a, a_stride, decay_ready, dt_bias, a_log, decay, state, cu_q, state_slot, y, heads, qk_heads, dk, dv, \
+               positions, rot_freq, rot)
     // short steps stage little, so that more CTAs are resident while their states stream in
 #define SOMI_LAUNCH_REC(TT, RR, DD)                                                               \
     if (max_rows > 0 && max_rows <= kRecBlockShort) { SOMI_LAUNCH_REC_B(TT, RR, DD, kRecBlockShort); } \
@@ -853,22 +897,24 @@ SOMI_API int somi_matrix_state_prepare(const void* q, const void* k, int dtype, 
                                        float q_scale, const float* a, long long a_stride,
                                        const float* dt_bias, const float* a_log, float* qn, float* kn,
                                        float* gd, int T, int heads, int qk_heads, int dk,
+                                       const int* positions, const double* rot_freq, int rot,
                                        cudaStream_t stream) {
     if (T <= 0) return 0;
     if (dk <= 0 || dk > 32 * kRecMaxPL || heads <= 0 || qk_heads <= 0 || heads % qk_heads ||
-        (a != nullptr && (dt_bias == nullptr || a_log == nullptr || gd == nullptr)))
+        (a != nullptr && (dt_bias == nullptr || a_log == nullptr || gd == nullptr)) || rot < 0 || (rot & 1) ||
+        rot > dk || (rot > 0 && (positions == nullptr || rot_freq == nullptr)))
         return SOMI_ERR_UNSUPPORTED;
     const dim3 grid((T + kRecPrepWarps - 1) / kRecPrepWarps, heads);
     if (dtype == SOMI_F32)
         launch_pdl(matrix_state_prepare_kernel<float>, grid, dim3(kRecPrepWarps * 32), 0, stream,
                    static_cast<const float*>(q), static_cast<const float*>(k), q_stride, k_stride,
                    act_silu, unit, unit_eps, q_scale, a, a_stride, dt_bias, a_log, qn, kn, gd, T, heads,
-                   qk_heads, dk);
+                   qk_heads, dk, positions, rot_freq, rot);
     else
         launch_pdl(matrix_state_prepare_kernel<__nv_bfloat16>, grid, dim3(kRecPrepWarps * 32), 0, stream,
                    static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k), q_stride,
                    k_stride, act_silu, unit, unit_eps, q_scale, a, a_stride, dt_bias, a_log, qn, kn, gd,
-                   T, heads, qk_heads, dk);
+                   T, heads, qk_heads, dk, positions, rot_freq, rot);
     return launch_status();
 }
 
@@ -877,7 +923,7 @@ SOMI_API int somi_group_rmsnorm_gate(const float* y, const void* gate, int g_dty
                                      int out_dtype, int T, int C, int groups, int gate_act,
                                      cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (groups <= 0 || C % groups || w_len <= 0) return SOMI_ERR_UNSUPPORTED;
+    if (groups <= 0 || C % groups || (weight != nullptr && w_len <= 0)) return SOMI_ERR_UNSUPPORTED;
     const int threads = threads_for(C / groups);
     if (C / groups <= kPartWarpMax) {                     // short parts: a warp each
         const long long parts = static_cast<long long>(T) * groups;

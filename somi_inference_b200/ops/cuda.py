@@ -640,20 +640,24 @@ class CudaOps:
         if trace.active():
             trace.note("xielu", 2 * out.numel() * out.element_size())
 
-    def head_product(self, x: torch.Tensor, w: torch.Tensor, heads_first: bool) -> torch.Tensor:
+    def head_product(self, x: torch.Tensor, w: torch.Tensor, heads_first: bool,
+                     out: torch.Tensor | None = None) -> torch.Tensor:
         """A product per head: y_h = x_h @ w_h^T with w [heads, N, K].
 
         `heads_first`: x is [T, heads, K] (a view of a [T, heads * K] projection) and y comes
         back as [heads, T, N]; otherwise x is [heads, T, K] and y is [T, heads, N], so that the
-        next projection reads [T, heads * N] without a copy.  float32: the engine's own product,
+        next projection reads [T, heads * N] without a copy.  x may be a view of wider rows; `out`
+        (heads_first only): a [heads, T, N] view that receives y.  float32: the engine's own product,
         batched over heads; bfloat16: the library's batched product."""
         H, N, K = w.shape
         if heads_first:
             T = x.shape[0]
             xs = x.transpose(0, 1)                               # [H, T, K] view
-            y = torch.empty((H, T, N), dtype=x.dtype, device=x.device)
+            y = torch.empty((H, T, N), dtype=x.dtype, device=x.device) if out is None else out
             ys = y
+            assert ys.shape == (H, T, N) and ys.stride(2) == 1 and ys.dtype == x.dtype
         else:
+            assert out is None
             T = x.shape[1]
             xs = x
             y = torch.empty((T, H, N), dtype=x.dtype, device=x.device)
@@ -675,18 +679,47 @@ class CudaOps:
                        detail=f"heads={H} M={T} N={N} K={K}")
         return y
 
-    def check_latent_geometry(self, heads: int, rank: int) -> None:
-        if not (1 <= rank <= 512 and 1 <= heads <= 65535):
-            raise KernelError(f"latent attention over a latent of {rank} elements with {heads} "
-                              "heads is not supported (latent up to 512)")
+    def check_latent_geometry(self, heads: int, rank: int, tail: int = 0) -> None:
+        if not (1 <= rank <= 512 and tail >= 0 and rank + tail <= 1024 and 1 <= heads <= 65535):
+            raise KernelError(f"latent attention over a latent of {rank} elements (and {tail} that only "
+                              f"the scores read) with {heads} heads is not supported (latent up to 512, "
+                              "rows up to 1024)")
 
-    def latent_attention(self, q, cache, batch, group, heads, rank, scale, window, sinks, out) -> None:
+    def latent_rotary_store(self, x, q_at: int, heads: int, q_dim: int, rot: int, c_at: int, rank: int,
+                            positions, inv_freq, neighbours: bool, weight, eps, slot_map, cache, qa) -> None:
+        """Rows of `x` hold, from column `q_at` on, query heads of q_dim + rot elements, and from
+        `c_at` on a latent of `rank` elements with a key part of `rot` behind it.  The token's cache
+        row [rank + rot] receives rmsnorm(latent) * weight and the turned key part, and
+        qa[:, :, rank:] ([heads, T, rank + rot]) every query's turned tail.  Pairs turn by position *
+        inv_freq[i] (float64): neighbours (2i, 2i + 1), or entries i and i + rot / 2."""
+        _check(positions, inv_freq, weight, slot_map, cache, qa)
+        if not (x.is_cuda and x.stride(1) == 1 and x.shape[1] >= max(q_at + heads * (q_dim + rot), c_at + rank + rot)):
+            raise KernelError("latent_rotary_store takes a device tensor with contiguous rows")
+        T = x.shape[0]
+        assert inv_freq.dtype == torch.float64 and inv_freq.numel() >= max(1, rot // 2)
+        assert qa.dtype == x.dtype and tuple(qa.shape) == (heads, T, rank + rot)
+        if slot_map is not None:
+            assert cache.dtype == x.dtype and cache.shape[1] == 1 and cache.shape[3] == rank + rot
+        rc = self.lib.somi_latent_rotary_store(
+            _ptr(x), _code(x), ctypes.c_longlong(x.stride(0)), ctypes.c_int(q_at), ctypes.c_int(heads),
+            ctypes.c_int(q_dim), ctypes.c_int(rot), ctypes.c_int(c_at), ctypes.c_int(rank),
+            ctypes.c_int(1 if neighbours else 0), _ptr(positions), _ptr(inv_freq), _ptr(weight),
+            _code(weight), ctypes.c_float(eps), _ptr(slot_map), _ptr(cache), _ptr(qa), ctypes.c_int(T),
+            self._stream())
+        self._done(rc, "latent_rotary_store")
+        if trace.active():
+            trace.note("latent_rotary_store", 2 * T * (heads * rot + rank + rot) * x.element_size())
+
+    def latent_attention(self, q, cache, batch, group, heads, rank, scale, window, sinks, out,
+                         tail: int = 0) -> None:
         """Attention of every token of the step over a cache of latents that serve as keys and
-        as values for every head (`q`, `out`: [heads, T, rank]; cache [pages, 1, page, rank]);
+        as values for every head (`q`, `out`: [heads, T, rank]; cache [pages, 1, page, rank]).
+        `tail`: elements behind the latent in q's and the cache's rows that only the scores read;
         `sinks`: float32 [heads] scores that join every softmax's denominator, or None."""
         _check(q, cache, out, group.block_table, sinks)
-        assert q.dtype == cache.dtype == out.dtype and q.shape == out.shape == (heads, q.shape[1], rank)
-        assert cache.shape[1] == 1 and cache.shape[3] == rank
+        wide = rank + tail
+        assert q.dtype == cache.dtype == out.dtype and q.shape == (heads, q.shape[1], wide)
+        assert out.shape == (heads, q.shape[1], rank) and cache.shape[1] == 1 and cache.shape[3] == wide
         assert sinks is None or (sinks.dtype == torch.float32 and sinks.numel() == heads)
         page_size = cache.shape[2]
         T = q.shape[1]
@@ -694,8 +727,8 @@ class CudaOps:
         n_decode = batch.num_requests - batch.num_prefill_requests
         win = int(window) if window else 0
         if (self.use_mma_latent and q.dtype == torch.bfloat16
-                and bool(self.lib.somi_latent_attention_mma_supported(ctypes.c_int(heads),
-                                                                      ctypes.c_int(rank)))):
+                and bool(self.lib.somi_latent_attention_mma_supported(
+                    ctypes.c_int(heads), ctypes.c_int(wide), ctypes.c_int(rank)))):
             # tensor cores: 16 tokens x 4 heads per CTA for prompt portions; all heads of a
             # single-token request per CTA, its keys in chunks whose partial sums are merged
             max_kv = group.width * page_size      # a bound that changes with the layout only
@@ -703,12 +736,12 @@ class CudaOps:
                 ctypes.c_int(max_kv), ctypes.c_int(win), ctypes.c_int(n_decode), ctypes.c_int(heads)))
             ws = self._scratch(n_decode * heads * splits * (rank + 2), q.device) if splits > 1 and n_decode else None
             rc = self.lib.somi_latent_attention_mma(
-                _ptr(q), ctypes.c_longlong(rank), ctypes.c_longlong(T * rank), _ptr(cache),
+                _ptr(q), ctypes.c_longlong(wide), ctypes.c_longlong(T * wide), _ptr(cache),
                 _ptr(group.block_table), ctypes.c_int(group.width), _ptr(batch.cu_q),
                 _ptr(batch.ctx_len), _ptr(tiles), ctypes.c_int(tiles.shape[0]),
                 ctypes.c_int(batch.num_prefill_requests), ctypes.c_int(batch.num_prefill_tokens),
                 ctypes.c_int(n_decode), ctypes.c_int(max_kv), ctypes.c_int(heads),
-                ctypes.c_int(rank), ctypes.c_int(page_size), ctypes.c_float(scale),
+                ctypes.c_int(wide), ctypes.c_int(rank), ctypes.c_int(page_size), ctypes.c_float(scale),
                 ctypes.c_int(win), _ptr(sinks), _ptr(out), ctypes.c_longlong(rank),
                 ctypes.c_longlong(T * rank), _ptr(ws), self._stream())
             self._done(rc, "latent_attention_mma")
@@ -716,15 +749,16 @@ class CudaOps:
             if trace.active():
                 moved, flops = self._attention_work(batch, 0, batch.num_requests, heads, 1, rank,
                                                     q.element_size(), win)
-                trace.note("latent_attention_mma", moved / 2 + heads * T * rank * q.element_size(), flops,
+                moved, flops = moved / 2 * (wide / rank), flops / 2 * (1 + wide / rank)
+                trace.note("latent_attention_mma", moved + heads * T * rank * q.element_size(), flops,
                            detail=f"splits={splits}" if n_decode else "")
             return
         rc = self.lib.somi_latent_attention_generic(
-            _ptr(q), _code(q), ctypes.c_longlong(rank), ctypes.c_longlong(T * rank), _ptr(cache),
+            _ptr(q), _code(q), ctypes.c_longlong(wide), ctypes.c_longlong(T * wide), _ptr(cache),
             _ptr(group.block_table), ctypes.c_int(group.width), _ptr(batch.cu_q),
             _ptr(batch.ctx_len), _ptr(tiles), ctypes.c_int(tiles.shape[0]),
             ctypes.c_int(batch.num_prefill_requests), ctypes.c_int(batch.num_prefill_tokens),
-            ctypes.c_int(n_decode), ctypes.c_int(heads), ctypes.c_int(rank),
+            ctypes.c_int(n_decode), ctypes.c_int(heads), ctypes.c_int(wide), ctypes.c_int(rank),
             ctypes.c_int(page_size), ctypes.c_float(scale), ctypes.c_int(int(window) if window else 0),
             _ptr(sinks), _ptr(out), ctypes.c_longlong(rank), ctypes.c_longlong(T * rank),
             self._stream())
@@ -732,7 +766,8 @@ class CudaOps:
         if trace.active():
             moved, flops = self._attention_work(batch, 0, batch.num_requests, heads, 1, rank,
                                                 q.element_size(), int(window) if window else 0)
-            trace.note("latent_attention_generic", moved / 2 + heads * T * rank * q.element_size(), flops)
+            moved, flops = moved / 2 * (wide / rank), flops / 2 * (1 + wide / rank)
+            trace.note("latent_attention_generic", moved + heads * T * rank * q.element_size(), flops)
 
     # ------------------------------- sandwich norms, convolutions, pair rotation, recurrence
     def embed_scaled(self, ids, table, scale: float, out) -> None:
@@ -1135,6 +1170,98 @@ class CudaOps:
                        + (out.numel() + (0 if extra is None else extra.numel())) * 4)
         return out
 
+    # ------------------------------- streams without pre-norms, averages over depth, turned values
+    def stream_update(self, x_in, x_out, delta, weight_b, eps_b, average, weight, eps, out, rows=None) -> None:
+        """r = x_in + rmsnorm(delta) * weight_b (no weight_b: x_in + delta; no delta: x_in); with
+        `average` = (start, results, n, coef) the record results[n - 1] = r and x = coef[0] * start +
+        sum of coef[j] * results[j - 1] over 1 <= j <= n (start float32 [N, H], results float32
+        [layers, N, H], coef float32 [n + 1]), else x = r.  x_out = x (float32; may be x_in), and,
+        where given, out = x in its dtype or, with `weight`, rmsnorm(x) * weight.  `delta`: [N, H] or
+        float32 [splits, N, H] partial sums added in order.  With `rows`, only those rows of `out`
+        are produced and neither x_out nor results are written."""
+        start, results, n, coef = average if average is not None else (None, None, 0, None)
+        _check(x_in, x_out, delta, weight_b, start, results, coef, weight, out, rows)
+        assert x_in.dtype == torch.float32 and (x_out is None or x_out.dtype == torch.float32)
+        N, H = x_in.shape
+        splits, stride = 1, 0
+        if delta is not None and delta.dim() == 3:
+            assert delta.dtype == torch.float32
+            splits, stride = delta.shape[0], delta.shape[1] * delta.shape[2]
+        if average is not None:
+            assert start.dtype == results.dtype == coef.dtype == torch.float32 and coef.numel() == n + 1
+            assert 1 <= n <= results.shape[0] and tuple(results.shape[1:]) == tuple(start.shape) == (N, H)
+        n_out = N if rows is None else rows.shape[0]
+        assert rows is not None or x_out is not None
+        rc = self.lib.somi_stream_update(
+            _ptr(x_in), _ptr(x_out), _ptr(delta), _code(delta) if delta is not None else _F32,
+            ctypes.c_int(splits), ctypes.c_longlong(stride), _ptr(weight_b),
+            _code(weight_b) if weight_b is not None else _F32, ctypes.c_float(eps_b), _ptr(start),
+            _ptr(results), ctypes.c_longlong(N * H), ctypes.c_int(n), _ptr(coef), _ptr(weight),
+            _code(weight) if weight is not None else _F32, ctypes.c_float(eps), _ptr(out),
+            _code(out) if out is not None else _F32, _ptr(rows), ctypes.c_int(n_out), ctypes.c_int(H),
+            ctypes.c_int(0 if rows is not None else 1), self._stream())
+        self._done(rc, "stream_update")
+        if trace.active():
+            e = n_out * H
+            moved = e * 4 * (1 if rows is not None or (delta is None and average is None and x_in is x_out) else 2)
+            if delta is not None:
+                moved += splits * e * delta.element_size()
+            if average is not None:
+                moved += e * 4 * (n + (1 if rows is None else 0))
+            if out is not None:
+                moved += e * out.element_size()
+            trace.note("stream_update", moved, detail=(f"average of {n + 1}" if average is not None else "")
+                       + (f" splits={splits}" if splits > 1 else ""))
+
+    def rownorm_rotary_store(self, qkv, positions, inv_freq, v_freq, nq, nkv, hd, vd, rotary_dim,
+                             neighbours: bool, q_weight, k_weight, eps, slot_map, kcache, vcache, turn=None) -> None:
+        """Rows of `qkv` hold nq query heads and nkv key heads of `hd` elements, then nkv value
+        heads of `vd`.  All query rows at once, and all key rows at once, pass an RMS norm with
+        `q_weight` [nq * hd] / `k_weight` [nkv * hd] (None: no norm); the pairs among the first
+        `rotary_dim` entries of query and key heads turn by position * inv_freq[i], and with `v_freq` the
+        pairs of every value head over its whole width by position * v_freq[m] (both float64).
+        Pairs: entries i and i + half, or `neighbours`.  Queries are rewritten in place; keys and
+        values go to their cache slots.  `turn`: float32 [T, vd / 2, 2], receives cosine and sine of
+        the value pairs' angles for `turn_back`."""
+        _check(positions, inv_freq, v_freq, slot_map, kcache, vcache, q_weight, k_weight, turn)
+        if not (qkv.is_cuda and qkv.stride(1) == 1 and qkv.shape[1] >= (nq + nkv) * hd + nkv * vd):
+            raise KernelError("rownorm_rotary_store takes a device tensor with contiguous rows")
+        assert inv_freq.dtype == torch.float64 and inv_freq.numel() >= max(1, rotary_dim // 2)
+        assert v_freq is None or (v_freq.dtype == torch.float64 and v_freq.numel() >= vd // 2)
+        assert (q_weight is None) == (k_weight is None)
+        assert q_weight is None or (q_weight.numel() == nq * hd and k_weight.numel() == nkv * hd
+                                    and q_weight.dtype == k_weight.dtype)
+        assert turn is None or (v_freq is not None and turn.dtype == torch.float32
+                                and tuple(turn.shape) == (qkv.shape[0], vd // 2, 2))
+        page_size = 1
+        if slot_map is not None:
+            assert kcache.dtype == qkv.dtype and vcache.dtype == qkv.dtype
+            assert kcache.shape[1] == nkv and kcache.shape[3] == hd and vcache.shape[3] == vd
+            page_size = kcache.shape[2]
+        rc = self.lib.somi_rownorm_rotary_store(
+            _ptr(qkv), _code(qkv), ctypes.c_longlong(qkv.stride(0)), _ptr(positions), _ptr(inv_freq),
+            _ptr(v_freq), ctypes.c_int(qkv.shape[0]), ctypes.c_int(nq), ctypes.c_int(nkv), ctypes.c_int(hd),
+            ctypes.c_int(vd), ctypes.c_int(rotary_dim), ctypes.c_int(1 if neighbours else 0), _ptr(q_weight),
+            _ptr(k_weight), _code(q_weight) if q_weight is not None else _F32, ctypes.c_float(eps),
+            _ptr(slot_map), _ptr(kcache), _ptr(vcache), ctypes.c_int(page_size), _ptr(turn), self._stream())
+        self._done(rc, "rownorm_rotary_store")
+        if trace.active():
+            n = qkv.shape[0] * ((nq + nkv) * hd + nkv * vd)
+            trace.note("rownorm_rotary_store", 2 * n * qkv.element_size())
+
+    def turn_back(self, x, turn, heads: int, vd: int, neighbours: bool = False) -> None:
+        """The pairs of every head of x [T, heads * vd] turned back in place by the angles whose
+        cosines and sines `turn` [T, vd / 2, 2] holds."""
+        _check(x, turn)
+        assert x.shape[1] == heads * vd and turn.dtype == torch.float32
+        assert tuple(turn.shape) == (x.shape[0], vd // 2, 2)
+        rc = self.lib.somi_turn_back(_ptr(x), _code(x), _ptr(turn), ctypes.c_longlong(x.shape[0]),
+                                     ctypes.c_int(heads), ctypes.c_int(vd), ctypes.c_int(1 if neighbours else 0),
+                                     self._stream())
+        self._done(rc, "turn_back")
+        if trace.active():
+            trace.note("turn_back", 2 * x.numel() * x.element_size() + turn.numel() * 4)
+
     # ------------------------------- side-by-side branches, matrix-state mixers, routers
     def add_scaled_rmsnorm(self, residual, a, scale_a, b, scale_b, mult: float, extra, w1, w2,
                            eps: float, out1, out2, rows=None) -> None:
@@ -1225,10 +1352,11 @@ class CudaOps:
     # a step in which some request has more rows than this has q, k and the decays made ready
     # once per row by a kernel of their own instead of once per group of state columns
     SCAN_PREPARE_ROWS = 16
+    SCAN_TURN_ROWS = 4          # the most rows a request may have where the scan itself rotates q and k
 
     def matrix_state_scan(self, q, k, v, state, batch, y, heads, qk_heads, dk, dv, *,
                           act_silu=False, unit_eps=None, q_scale=1.0, beta=None, decay_logits=None,
-                          dt_bias=None, a_log=None, decay=None, prepare=None) -> None:
+                          dt_bias=None, a_log=None, decay=None, rotary=None, prepare=None) -> None:
         """Per request and head a float32 state S [dk, dv] in `state` [slots, heads, dv, dk] (a
         head's matrix column by column), continued over the request's rows of this step:
             S <- g * S;  u = v, or with `beta` u = sigmoid(beta) * (v - S^T k);  S <- S + k u^T;
@@ -1237,7 +1365,9 @@ class CudaOps:
         dt_bias)) (`decay_logits` float32 [T, heads * dk], rows may lie further apart).  q, k
         ([T, qk_heads * dk]) and v ([T, heads * dv]) may be views of wider rows; `act_silu`: they
         pass SiLU as they are read; `unit_eps`: q and k are divided by sqrt(sum of squares + it);
-        q is multiplied by `q_scale` either way.  y: float32 [T, heads * dv].  `prepare` (None: by the
+        q is multiplied by `q_scale` either way.  `rotary` = (positions [T], float64 inv_freq, dims): the
+        pairs (i, i + dims / 2) of every q and k head turn by position * inv_freq[i] first.  y: float32
+        [T, heads * dv].  `prepare` (None: by the
         step's longest request) only chooses where q, k and g are computed; y is the same."""
         _check(state, y, dt_bias, a_log, decay)
         for t in (q, k, v, beta, decay_logits):
@@ -1251,6 +1381,12 @@ class CudaOps:
         max_rows = int(getattr(batch, "max_q_len", 0) or 0)
         if prepare is None:
             prepare = max_rows > self.SCAN_PREPARE_ROWS
+        pos, freq, rot = rotary if rotary is not None else (None, None, 0)
+        if rot:
+            _check(pos, freq)
+            assert pos.dtype == torch.int32 and freq.dtype == torch.float64 and freq.numel() >= rot // 2
+            # the scan turns q and k itself only in steps of a few rows
+            prepare = prepare or not 0 < max_rows <= self.SCAN_TURN_ROWS
         act, unit, ready = (3 if act_silu else 0), (0 if unit_eps is None else 1), 0
         vb_code = _code(v)
         if prepare:
@@ -1265,12 +1401,14 @@ class CudaOps:
                 ctypes.c_float(q_scale), _ptr(decay_logits),
                 ctypes.c_longlong(decay_logits.stride(0) if decay_logits is not None else 0),
                 _ptr(dt_bias), _ptr(a_log), _ptr(qn), _ptr(kn), _ptr(gd), ctypes.c_int(T),
-                ctypes.c_int(heads), ctypes.c_int(qk_heads), ctypes.c_int(dk), self._stream())
+                ctypes.c_int(heads), ctypes.c_int(qk_heads), ctypes.c_int(dk), _ptr(pos), _ptr(freq),
+                ctypes.c_int(rot), self._stream())
             self._done(rc, "matrix_state_prepare")
             if trace.active():
                 trace.note("matrix_state_prepare", 2 * n * (q.element_size() + 4) + 2 * n_g * 4)
             q, k, decay_logits = qn, kn, gd
             act, unit, ready, q_scale = act & 2, 0, 1, 1.0      # q is scaled already
+            pos, freq, rot = None, None, 0                      # and q and k are turned
         rc = self.lib.somi_matrix_state_scan(
             _ptr(q), _ptr(k), _ptr(v), _code(q), vb_code, ctypes.c_longlong(q.stride(0)),
             ctypes.c_longlong(k.stride(0)), ctypes.c_longlong(v.stride(0)),
@@ -1283,7 +1421,7 @@ class CudaOps:
             _ptr(dt_bias), _ptr(a_log), _ptr(decay), _ptr(state), _ptr(batch.cu_q),
             _ptr(batch.state_slot), _ptr(y), ctypes.c_int(batch.num_requests), ctypes.c_int(heads),
             ctypes.c_int(qk_heads), ctypes.c_int(dk), ctypes.c_int(dv),
-            ctypes.c_int(max_rows), self._stream())
+            ctypes.c_int(max_rows), _ptr(pos), _ptr(freq), ctypes.c_int(rot), self._stream())
         self._done(rc, "matrix_state_scan")
         if trace.active():
             T = q.shape[0]
@@ -1296,18 +1434,19 @@ class CudaOps:
 
     def group_rmsnorm_gate(self, y, gate, weight, eps, groups, out, gate_act: str = "sigmoid") -> None:
         """out = rmsnorm over each of `groups` equal parts of y (float32), times weight (as long
-        as a row, or as a part and then shared by the parts), times sigmoid(gate) where there is
+        as a row, or as a part and then shared by the parts; None: no weight), times sigmoid(gate) where there is
         a gate ([T, C], rows may lie further apart); `gate_act` "silu": times silu(gate) instead."""
         _check(y, weight, out)
         if gate is not None and not (gate.is_cuda and gate.stride(1) == 1 and gate.shape == y.shape):
             raise KernelError("group_rmsnorm_gate takes a gate with contiguous rows")
         assert y.dtype == torch.float32
         C = y.shape[1]
-        assert weight.numel() in (C, C // groups)
+        assert weight is None or weight.numel() in (C, C // groups)
         rc = self.lib.somi_group_rmsnorm_gate(
             _ptr(y), _ptr(gate), ctypes.c_int(_code(gate) if gate is not None else _F32),
-            ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _ptr(weight), _code(weight),
-            ctypes.c_int(weight.numel()), ctypes.c_float(eps), _ptr(out), _code(out),
+            ctypes.c_longlong(gate.stride(0) if gate is not None else 0), _ptr(weight),
+            _code(weight) if weight is not None else _F32,
+            ctypes.c_int(weight.numel() if weight is not None else 0), ctypes.c_float(eps), _ptr(out), _code(out),
             ctypes.c_int(y.shape[0]), ctypes.c_int(C), ctypes.c_int(groups),
             ctypes.c_int({"sigmoid": 0, "silu": 1}[gate_act]), self._stream())
         self._done(rc, "group_rmsnorm_gate")
@@ -1351,13 +1490,14 @@ class CudaOps:
             trace.note("relu2", 2 * x.numel() * x.element_size())
 
     def moe_router_select(self, logits, correction, count: int, keep: int, top: int,
-                          over_chosen: bool = False):
+                          over_chosen: bool = False, sigmoid: bool = False, group_best: int = 1):
         """logits float32 [T, n] -> (chosen int32 [T, top], weight float32 [T, top]): softmax over
         the n outputs; the choice is made on softmax + correction (None: the softmax) among the
         members of the `keep` best of `count` equal groups of neighbours (a group's score is its
         best member's; count <= 1: no groups); the weights are the chosen outputs' softmax.
         `over_chosen`: the `top` largest logits are chosen (no correction, no groups) and the
-        weights are the softmax over the chosen logits only."""
+        weights are the softmax over the chosen logits only.  `sigmoid`: sigmoids of the logits take the
+        softmax's place; `group_best` 2: a group's score is the sum of its two best members'."""
         _check(logits, correction)
         assert logits.dtype == torch.float32 and (correction is None or correction.dtype == torch.float32)
         T, n = logits.shape
@@ -1367,7 +1507,9 @@ class CudaOps:
                                              _ptr(correction), ctypes.c_int(T), ctypes.c_int(n),
                                              ctypes.c_int(count), ctypes.c_int(keep), ctypes.c_int(top),
                                              _ptr(chosen), _ptr(weight),
-                                             ctypes.c_int(1 if over_chosen else 0), self._stream())
+                                             ctypes.c_int(1 if over_chosen else 0),
+                                             ctypes.c_int(1 if sigmoid else 0), ctypes.c_int(group_best),
+                                             self._stream())
         self._done(rc, "moe_router_select")
         if trace.active():
             trace.note("moe_router_select", T * (n * 4 + top * 8))
@@ -1448,12 +1590,14 @@ class CudaOps:
 
     def skinny_gemm(self, x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None,
                     mode: int = 0, splits: int = 1, deep_ring: bool = False,
-                    act: torch.Tensor | None = None, n_act: int = 0):
+                    act: torch.Tensor | None = None, n_act: int = 0, gated=(float("inf"), 1.0, 0.0)):
         """x[M, K] @ w[N, K]^T on tcgen05 tensor cores for M <= 64.
 
         mode GEMM_BF16 -> bf16 [M, N] (+ bias); GEMM_F32 -> float32 [M, N];
         GEMM_PARTIAL_F32 -> float32 [splits', M, N] partial sums over ranges of K (bias in the
-        first); GEMM_SWIGLU -> bf16 [M, N / 2] = silu(even rows) * odd rows of w;
+        first); GEMM_SWIGLU -> bf16 [M, N / 2]: with g the even rows' and u the odd rows' features and
+        `gated` = (limit, alpha, shift), g' * sigmoid(alpha * g') * (u' + shift) where g' = min(g, limit)
+        and u' = u within +-limit (the default is silu(g) * u);
         GEMM_XIELU_SIDE -> (bf16 [M, n_act] = xIELU of the first n_act features with the two
         numbers of `act` (float32), bf16 [M, N - n_act] = the other features), bias added to both.
         """
@@ -1487,13 +1631,15 @@ class CudaOps:
                 ctypes.c_int(box), ctypes.c_int(M), ctypes.c_int(N), ctypes.c_int(K),
                 ctypes.c_int(1), ctypes.c_int(mode), _ptr(bias),
                 _code(bias) if bias is not None else _F32, _ptr(out), _ptr(out2),
-                ctypes.c_int(n_act), _ptr(act), ctypes.c_int(1 if deep_ring else 0), self._stream())
+                ctypes.c_int(n_act), _ptr(act), *(ctypes.c_float(v) for v in self._gated(gated)),
+                ctypes.c_int(1 if deep_ring else 0), self._stream())
         else:
             rc = self.lib.somi_skinny_gemm(
                 ctypes.c_void_p(self._gemm_map(w, 128)), ctypes.c_void_p(self._gemm_map(x, box)),
                 ctypes.c_int(box), ctypes.c_int(M), ctypes.c_int(N), ctypes.c_int(K),
                 ctypes.c_int(splits), ctypes.c_int(mode), _ptr(bias),
                 _code(bias) if bias is not None else _F32, _ptr(out),
+                *(ctypes.c_float(v) for v in self._gated(gated)),
                 ctypes.c_int(1 if deep_ring else 0), self._stream())
         self._done(rc, "skinny_gemm")
         if trace.active():

@@ -32,6 +32,8 @@ Interfaces (duck-typed; the classes below only document them):
 * Stream part:   `forward(residual, pending, start) -> float32 [T, H]`: the stream that replaces
                  `residual` in front of a run whose `RunSpec.remix` names the part; `pending` is
                  what the run before left to be added (or None), `start` the embedding's output.
+                 A part that `RunSpec.average` names answers `behind(pending, start, results, index)
+                 -> DepthAverage` instead.
 * Layer extra:   whatever its arrangement calls; `declare(params)` and `__init__(params,
                  tensors, ctx)` like every part.
 """
@@ -154,6 +156,30 @@ class BranchSum:
 
     a: torch.Tensor
     b: torch.Tensor | None = None
+
+
+@dataclass
+class StreamStart:
+    """The stream begins as these float32 rows [T, H], which stay as they are: the first norm reads
+    them and writes the stream (a schedule that needs the embedding's output later on)."""
+
+    rows: torch.Tensor
+
+
+@dataclass
+class DepthAverage:
+    """What a run behind which the stream is averaged over depth hands to the next norm: what is
+    pending (None, a tensor or partial sums, or a `NormedDelta`), the embedding's output X_0
+    (float32 [T, H]), the record of the runs' results (float32 [runs, T, H]: X_j lies at j - 1), this
+    run's number n (from 1 on) and float32 coefficients [n + 1].  The next norm adds what is pending
+    to the stream, which is the result X_n, stores it and replaces the stream by the sum over j of
+    coefficient j times X_j before it goes on."""
+
+    pending: Any
+    start: torch.Tensor
+    results: torch.Tensor
+    n: int
+    coefficients: torch.Tensor
 
 
 def with_extra_rows(pending, rows: torch.Tensor):

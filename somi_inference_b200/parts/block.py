@@ -38,7 +38,7 @@ class SandwichNormBlock:
     """A norm before and a norm behind each branch:
         x = x + norm_b(mixer(norm_a(x)));  x = x + norm_d(feed_forward(norm_c(x)))
     Norms: `mixer`, `mixer_post`, and with a feed-forward `feed_forward`, `feed_forward_post`.  The
-    post norms must be RMS norms: their weight and eps travel with the branch's result as a
+    norms in front may be "none": the branch then reads the stream itself.  The post norms must be RMS norms: their weight and eps travel with the branch's result as a
     `NormedDelta`, and the next norm's kernel normalises the branch, adds it to the residual
     stream and normalises that, all in float32."""
 

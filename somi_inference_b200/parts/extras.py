@@ -16,7 +16,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import BranchSum, BuildContext, StateNeeds, TensorDecl, names_of
+from .base import BranchSum, BuildContext, DepthAverage, StateNeeds, TensorDecl, names_of
 from .linear import Linear
 from .registry import LAYER_EXTRAS, STREAM_PARTS
 
@@ -90,6 +90,28 @@ class Constant:
 
     def __init__(self, params, tensors, ctx: BuildContext) -> None:
         self.value = float(params["value"])
+
+
+@STREAM_PARTS.register("depth_average")
+class DepthAverageWeights:
+    """A learned weighted sum over depth that replaces the stream behind a run:
+        x <- sum_(j <= n) a_j X_j,     X_0 the embedding's output, X_j the result of run j (from 1 on)
+    `count` = n + 1 coefficients for run n.  The sum is float32 and is made by the next norm's kernel,
+    together with what the run left pending."""
+
+    @staticmethod
+    def declare(params) -> list[TensorDecl]:
+        return [TensorDecl(names_of(params)["weight"], (int(params["count"]),), matrix=False)]
+
+    def __init__(self, params, tensors, ctx: BuildContext) -> None:
+        self.coefficients = tensors[names_of(params)["weight"]].float().contiguous()
+
+    def behind(self, pending, start: torch.Tensor, results: torch.Tensor, index: int) -> DepthAverage:
+        """`index`: the run's place in the schedule, from 0 on."""
+        if self.coefficients.numel() != index + 2:
+            raise ValueError(f"an average over depth behind run {index} takes {index + 2} coefficients, "
+                             f"not {self.coefficients.numel()}")
+        return DepthAverage(pending, start, results, index + 1, self.coefficients)
 
 
 @STREAM_PARTS.register("embedding_remix")

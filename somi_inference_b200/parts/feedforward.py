@@ -15,6 +15,37 @@ from .linear import Linear
 from .registry import FEED_FORWARDS
 
 
+
+@FEED_FORWARDS.register("clamped_glu")
+class ClampedGLU:
+    """y = W_down (g sigmoid(alpha g) (u + shift)), g = min(W_gate h, limit), u = W_up h within
+    +-limit.  The activation is float32; a step of few tokens makes it in the product's epilogue."""
+
+    graph_safe = True
+
+    @staticmethod
+    def declare(params) -> list[TensorDecl]:
+        return SwiGLU.declare(params)
+
+    def __init__(self, params, tensors, ctx: BuildContext) -> None:
+        n = names_of(params)
+        self.ctx = ctx
+        gate, up = tensors[n["gate_weight"]], tensors[n["up_weight"]]
+        self.gate_up = Linear(torch.stack([gate, up], dim=1).reshape(2 * gate.shape[0], -1).contiguous(),
+                              None, ctx.ops)
+        self.down = Linear(tensors[n["down_weight"]], None, ctx.ops)
+        self.gated = (float(params["limit"]), float(params["alpha"]), float(params["shift"]))
+        if not self.gated[0] > 0.0:
+            raise ValueError("the limit of a clamped activation must be positive")
+
+    def forward(self, x: torch.Tensor, batch) -> torch.Tensor:
+        act = self.gate_up.swiglu(x, self.gated)
+        if act is None:
+            act = self.ctx.ops.clamped_gate_up(self.gate_up(x), *self.gated)
+        partial = self.down.partial_sums(act)
+        return partial if partial is not None else self.down(act)
+
+
 @FEED_FORWARDS.register("swiglu")
 class SwiGLU:
     graph_safe = True     # launches kernels only; nothing is decided on the host per step

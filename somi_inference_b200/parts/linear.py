@@ -58,11 +58,12 @@ class Linear:
         return ops.skinny_gemm(x, self.weight, self.bias, ops.GEMM_PARTIAL_F32,
                                splits=ops.skinny_splits(x.shape[0], self.out_features, self.in_features))
 
-    def swiglu(self, x: torch.Tensor) -> torch.Tensor | None:
-        """silu(gate) * up for a weight whose rows alternate gate, up; None when not available."""
+    def swiglu(self, x: torch.Tensor, gated=(float("inf"), 1.0, 0.0)) -> torch.Tensor | None:
+        """silu(gate) * up, or the gated activation (limit, alpha, shift), for a weight whose rows
+        alternate gate, up; None when not available."""
         if not self.skinny(x):
             return None
-        return self.ops.skinny_gemm(x, self.weight, None, self.ops.GEMM_SWIGLU)
+        return self.ops.skinny_gemm(x, self.weight, None, self.ops.GEMM_SWIGLU, gated=gated)
 
     def xielu_side(self, x: torch.Tensor, act: torch.Tensor, n_act: int):
         """(xIELU of the first `n_act` output features, the other features), bias added to both,

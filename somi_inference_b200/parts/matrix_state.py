@@ -17,8 +17,8 @@ H heads over G query/key heads (head i reads query/key head i // (H / G)):
     M <- decay * M + k v^T;  o = M^T q
     out = Wo (rmsnorm_over_all_heads(o) * norm * sigmoid(Wg h))
 
-`gated_linear_attention` (at the end of the file): a decay per key channel and token from a
-sigmoid, no correction, a SiLU gate.
+`gated_linear_attention`: a decay per key channel and token from a sigmoid, no correction, a SiLU
+gate.  `retention` (at the end of the file): rotated queries and keys, a constant decay per head.
 
 Products run in the compute dtype with float32 accumulation; unit norms, beta, the decays with
 their softplus and exponentials, the recurrence, the norms and the gates' sigmoids are float32 in
@@ -32,6 +32,7 @@ import torch
 
 from .base import BuildContext, CacheNeeds, StateNeeds, TensorDecl, names_of
 from .linear import Linear
+from .position import rotary_frequencies
 from .registry import MIXERS
 
 
@@ -253,5 +254,77 @@ class GatedLinearAttentionMixer:
         gated = torch.empty((T, self.inner), dtype=x.dtype, device=x.device)
         ops.group_rmsnorm_gate(y, proj[:, 2 * w + self.inner:], self.norm_weight, self.eps,
                                self.heads, gated, gate_act="silu")
+        partial = self.out.partial_sums(gated)
+        return partial if partial is not None else self.out(gated)
+
+
+@MIXERS.register("retention")
+class RetentionMixer:
+    """Linear attention with a constant decay per head and rotary positions, without a denominator:
+
+        q = Wq h, k = Wk h, v = Wv h                                  (heads x key / value width)
+        q, k: entry i < dims / 2 of a head is paired with entry i + dims / 2, the pair at position p
+              turns by p * base^(-2i / dims), entries from dims on pass; k then times `k_scale`
+        M <- decay_head * M + k v^T;  o = M^T q
+        out = Wo (o per head over its root mean square * silu(Wg h))        (no weight)
+
+    One factor for all of k is the same factor for o, so the kernel applies it with q.  Rotated q
+    and k, the recurrence, the norm and the gate's SiLU are float32: the scan's kernels rotate as
+    they read the projection."""
+
+    graph_safe = True
+    STATE = "retention_state"
+
+    @staticmethod
+    def declare(params) -> list[TensorDecl]:
+        n = names_of(params)
+        hidden, H = int(params["hidden_size"]), int(params["heads"])
+        d, dv = int(params["key_dim"]), int(params["value_dim"])
+        return [TensorDecl(n["q_weight"], (H * d, hidden)), TensorDecl(n["k_weight"], (H * d, hidden)),
+                TensorDecl(n["v_weight"], (H * dv, hidden)), TensorDecl(n["gate_weight"], (H * dv, hidden)),
+                TensorDecl(n["o_weight"], (hidden, H * dv))]
+
+    def __init__(self, params, tensors, ctx: BuildContext) -> None:
+        n = names_of(params)
+        self.ctx = ctx
+        self.heads = int(params["heads"])
+        self.key_dim, self.value_dim = int(params["key_dim"]), int(params["value_dim"])
+        ctx.ops.check_matrix_state_geometry(self.heads, self.heads, self.key_dim, self.value_dim)
+        decay = [float(v) for v in params["decay"]]
+        if len(decay) != self.heads:
+            raise ValueError(f"{len(decay)} decays for {self.heads} heads")
+        self.decay = torch.tensor(decay, dtype=torch.float32, device=ctx.device)
+        rotary = params.get("rotary") or {}
+        self.rotary_dim = int(rotary.get("dims", 0))
+        if self.rotary_dim % 2 or self.rotary_dim > self.key_dim:
+            raise ValueError("rotary dims must be even and at most the key width")
+        inv, magnitude = rotary_frequencies(rotary)
+        self.inv_freq = inv.to(ctx.device)
+        self.eps = float(params["eps"])
+        self.k_scale = float(params.get("k_scale", 1.0)) * magnitude * magnitude
+        self.qk_width = self.heads * self.key_dim
+        self.inner = self.heads * self.value_dim
+        self.proj = Linear(torch.cat([tensors[n["q_weight"]], tensors[n["k_weight"]],
+                                      tensors[n["v_weight"]], tensors[n["gate_weight"]]], 0).contiguous(),
+                           None, ctx.ops)
+        self.out = Linear(tensors[n["o_weight"]], None, ctx.ops)
+
+    def cache_needs(self) -> CacheNeeds:
+        return CacheNeeds(paged=None, state=StateNeeds(
+            {self.STATE: ((self.heads, self.value_dim, self.key_dim), torch.float32)}))
+
+    def forward(self, x: torch.Tensor, batch, cache, owns_cache: bool) -> torch.Tensor:
+        ops = self.ctx.ops
+        T, w = x.shape[0], self.qk_width
+        proj = self.proj(x)                                     # [T, q | k | v | gate logits]
+        y = torch.empty((T, self.inner), dtype=torch.float32, device=x.device)
+        ops.matrix_state_scan(proj[:, :w], proj[:, w:2 * w], proj[:, 2 * w:2 * w + self.inner],
+                              cache.state[self.STATE], batch, y, self.heads, self.heads,
+                              self.key_dim, self.value_dim, q_scale=self.k_scale, decay=self.decay,
+                              rotary=((batch.positions, self.inv_freq, self.rotary_dim)
+                                      if self.rotary_dim else None))
+        gated = torch.empty((T, self.inner), dtype=x.dtype, device=x.device)
+        ops.group_rmsnorm_gate(y, proj[:, 2 * w + self.inner:], None, self.eps, self.heads, gated,
+                               gate_act="silu")
         partial = self.out.partial_sums(gated)
         return partial if partial is not None else self.out(gated)

@@ -13,7 +13,7 @@ from __future__ import annotations
 import torch
 
 from ..config.spec import LayerSpec, ModelSpec
-from .base import BuildContext, CacheNeeds, StateNeeds, TensorDecl, with_extra_rows
+from .base import BuildContext, CacheNeeds, StateNeeds, StreamStart, TensorDecl, with_extra_rows
 from .registry import (ARRANGEMENTS, EMBEDDINGS, FEED_FORWARDS, HEADS, LAYER_EXTRAS, MIXERS,
                        NORMS, STREAM_PARTS)
 
@@ -107,6 +107,14 @@ class Decoder:
         # is written by the norms from the first run on
         start = (residual.clone() if any(run.add_embedding or run.remix is not None
                                          for run in self.schedule) else None)
+        results = None
+        if any(run.average is not None for run in self.schedule):
+            # an average over depth reads the embedding's output and every run's result: the first
+            # norm starts the stream in rows of its own, and the results are recorded beside it
+            start, residual = residual, torch.empty_like(residual)
+            pending = StreamStart(start)
+            results = torch.empty((len(self.schedule), *start.shape), dtype=torch.float32,
+                                  device=start.device)
         for i, run in enumerate(self.schedule):
             if run.add_embedding:
                 pending = with_extra_rows(pending, start)
@@ -117,6 +125,8 @@ class Decoder:
                 pending = None
             pending = self.layers[run.layer].forward(residual, pending, batch, cache.view(i),
                                                      run.cache_of is None)
+            if run.average is not None:
+                pending = self.stream_parts[run.average].behind(pending, start, results, i)
         if batch.logit_rows.shape[0] == 0:
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32,
                                device=residual.device)

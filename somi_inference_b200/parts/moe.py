@@ -115,7 +115,8 @@ class RoutedMoE:
         experts without tensors: expert(h) = h
         y = sum of weight * expert(h) over the chosen
 
-    Two parameters change the form.  `weights` = "softmax_chosen": the `top` largest logits are
+    Parameters change the form.  `scores` = "sigmoid": s = sigmoid(W_router h) per output.  `groups.best`
+    = 2: a group's score is the sum of its two best choices.  `weights` = "softmax_chosen": the `top` largest logits are
     chosen (no correction, no groups) and the weights are the softmax over the chosen logits only.
     `activation` (a name of the kernel table's `ACTIVATIONS`, e.g. "gelu"): experts without a gate,
     expert(h) = W_down act(W_up h), and no gate tensors.
@@ -153,7 +154,14 @@ class RoutedMoE:
         self.act = params.get("activation")
         if self.act is not None and self.act not in ctx.ops.ACTIVATIONS:
             raise ValueError(f"unknown activation {self.act!r}; known: {sorted(ctx.ops.ACTIVATIONS)}")
+        scores = params.get("scores", "softmax")
+        if scores not in ("softmax", "sigmoid") or (self.over_chosen and scores != "softmax"):
+            raise ValueError(f"unknown router scores {scores!r} (kinds: 'softmax', 'sigmoid')")
+        self.sigmoid = scores == "sigmoid"
         groups = params.get("groups") or {}
+        self.group_best = int(groups.get("best", 1))
+        if self.group_best not in (1, 2):
+            raise ValueError("a group's score is made of its one or two best members")
         self.group_count = int(groups.get("count", 1))
         self.group_keep = int(groups.get("keep", self.group_count))
         if self.experts < 1 or not 1 <= self.top <= self.outputs:
@@ -180,7 +188,8 @@ class RoutedMoE:
         ops, top, E = self.ctx.ops, self.top, self.experts
         logits = self.router.to_float32(x)
         chosen, weight = ops.moe_router_select(logits, self.correction, self.group_count,
-                                               self.group_keep, top, over_chosen=self.over_chosen)
+                                               self.group_keep, top, over_chosen=self.over_chosen,
+                                               sigmoid=self.sigmoid, group_best=self.group_best)
         n_entries = x.shape[0] * top
         if ops.moe_gemv_supported(n_entries, x.shape[1], x.dtype) and self.w_down.shape[2] % 8 == 0:
             act = ops.moe_gemv(x, self.w_gate_up, None, chosen, per_token=True, gated=self.gated,

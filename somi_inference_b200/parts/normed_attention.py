@@ -1,12 +1,18 @@
-"""Attention whose queries and keys pass an RMS norm per head before they are rotated.
+"""Attention whose queries and keys pass an RMS norm (per head, or over the whole projection) before
+they are rotated.
 
 Per token, with h the mixer's input:
     q = Wq h + bq, k = Wk h + bk, v = Wv h + bv                    (`qkv_bias`)
     q, k: every head divided by its root mean square over the head (eps inside the root) and
-          multiplied by a weight of the head's width that all heads share     (`head_norm`)
+          multiplied by a weight of the head's width that all heads share     (`head_norm`);
+          or all query rows at once, and all key rows at once, over their root mean square, times
+          a weight as long as they are                                         (`row_norm`)
     q, k: entry i < dims / 2 of a head is paired with entry i + dims / 2; the pair of the token at
           position p turns by p * base^(-2i / dims); entries from `dims` on pass      (`rotary`;
           its `scaling` changes the frequencies: `position.rotary_frequencies`)
+    v: with `turn_values` entry m < value width / 2 of a value head is paired with entry m + half and the
+          pair turns by p * base^(-2m / value width); it is cached so, and every head's output is
+          turned back by its query's position (so a value arrives turned by its distance)
     scores q.k * scale, then cap * tanh(score / cap) where there is a `softcap`, over the keys the
           mask leaves: all earlier ones, or the token's own and the `size` - 1 before it
           (`mask` = {"kind": "window", "size"}); softmax, with `sink` = "zero" one more term
@@ -52,6 +58,9 @@ class NormedAttentionMixer:
         if params.get("head_norm"):
             decl += [TensorDecl(n["q_norm"], (d,), init="ones", matrix=False),
                      TensorDecl(n["k_norm"], (d,), init="ones", matrix=False)]
+        if params.get("row_norm"):
+            decl += [TensorDecl(n["q_norm"], (heads * d,), init="ones", matrix=False),
+                     TensorDecl(n["k_norm"], (kv_heads * d,), init="ones", matrix=False)]
         if params.get("head_gate"):
             decl.append(TensorDecl(n["gate_weight"], (heads, hidden)))
         if params.get("sink") == "learned":
@@ -83,6 +92,18 @@ class NormedAttentionMixer:
             raise ValueError("rotary dims must be even and at most the key width")
         inv, self.magnitude = rotary_frequencies(rotary)
         self.inv_freq = inv.to(ctx.device)
+        # norms over whole rows and turned values have a kernel of their own
+        self.row_norm, turn_values = bool(params.get("row_norm")), bool(params.get("turn_values"))
+        self.by_rows = self.row_norm or turn_values
+        if self.by_rows and (params.get("head_norm") or self.magnitude != 1.0):
+            raise ValueError("norms over whole rows and turned values do not go with norms per head "
+                             "or a rotation with a magnitude")
+        self.value_freq = None
+        if turn_values:
+            if self.value_dim % 2:
+                raise ValueError("turned values need an even value width")
+            vf, _ = rotary_frequencies({"dims": self.value_dim, "base": rotary["base"]})
+            self.value_freq = vf.to(ctx.device)
         self.softcap = float(params["softcap"]) if params.get("softcap") else None
         sink = params.get("sink")
         if sink not in (None, "zero", "learned"):
@@ -109,8 +130,9 @@ class NormedAttentionMixer:
             if bias is not None:
                 bias = torch.cat([bias, torch.zeros(self.heads + pad, dtype=bias.dtype, device=bias.device)])
         self.proj = Linear(torch.cat(weights, 0).contiguous(), bias, ctx.ops)
-        self.q_norm = tensors[n["q_norm"]] if params.get("head_norm") else None
-        self.k_norm = tensors[n["k_norm"]] if params.get("head_norm") else None
+        normed = params.get("head_norm") or self.row_norm
+        self.q_norm = tensors[n["q_norm"]] if normed else None
+        self.k_norm = tensors[n["k_norm"]] if normed else None
         self.out = Linear(tensors[n["o_weight"]],
                           tensors[n["o_bias"]].float() if params.get("o_bias") else None, ctx.ops)
 
@@ -123,15 +145,27 @@ class NormedAttentionMixer:
         ops, paged = self.ctx.ops, cache.paged
         qkv = self.proj(x)
         group = batch.groups[paged.group]
-        ops.headnorm_rotary_store(qkv, batch.positions, self.inv_freq, self.heads, self.kv_heads,
-                                  self.key_dim, self.value_dim, self.rotary_dim, self.q_norm,
-                                  self.k_norm, self.eps, group.slot_map if owns_cache else None,
-                                  paged.keys, paged.values, magnitude=self.magnitude)
+        turn = None
+        if self.by_rows:
+            if self.value_freq is not None:
+                turn = torch.empty((x.shape[0], self.value_dim // 2, 2), dtype=torch.float32, device=x.device)
+            ops.rownorm_rotary_store(qkv, batch.positions, self.inv_freq, self.value_freq, self.heads,
+                                     self.kv_heads, self.key_dim, self.value_dim, self.rotary_dim, False,
+                                     self.q_norm, self.k_norm, self.eps,
+                                     group.slot_map if owns_cache else None, paged.keys, paged.values,
+                                     turn=turn)
+        else:
+            ops.headnorm_rotary_store(qkv, batch.positions, self.inv_freq, self.heads, self.kv_heads,
+                                      self.key_dim, self.value_dim, self.rotary_dim, self.q_norm,
+                                      self.k_norm, self.eps, group.slot_map if owns_cache else None,
+                                      paged.keys, paged.values, magnitude=self.magnitude)
         out = torch.empty((x.shape[0], self.heads * self.value_dim), dtype=x.dtype, device=x.device)
         ops.paged_attention(qkv, paged.keys, paged.values, batch, group, self.heads, self.kv_heads,
                             self.key_dim, self.scale, self.window, out, storage=paged.storage,
                             value_dim=self.value_dim,
                             gate=qkv[:, self.gate_at:self.gate_at + self.heads] if self.head_gate else None,
                             gate_per_head=self.head_gate, softcap=self.softcap, sinks=self.sinks)
+        if turn is not None:
+            ops.turn_back(out, turn, self.heads, self.value_dim)
         partial = self.out.partial_sums(out)
         return partial if partial is not None else self.out(out)
