@@ -8,6 +8,7 @@
     python bench.py --arch dapozen --only decode|prefill [...]   the same shapes with Dapozen layers
     python bench.py --arch poselorn --only decode|prefill [...]  the same shapes with Poselorn layers
     python bench.py --arch gikarax --only decode|prefill [...]   the same shapes with Gikarax layers
+    python bench.py --arch dosuvik --only decode|prefill [...]   the same shapes with Dosuvik layers
 
 A step is one decode step of the whole engine: 8 requests with 2,048 cached tokens each,
 random bfloat16 weights, one new token per request (batch layout upload, all layers, head,
@@ -83,6 +84,13 @@ POSELORN = dict(window=8192, taps=4, rank=128, experts=16, identity=4, top=3, gr
 # latents are Digosun's; the window is longer than the timed contexts (the attention reads what
 # the Qwen2 layer reads); the linear attention has the shape's heads at the same widths.
 GIKARAX = dict(window=8192, softcap=30.0, rank=128, tau=8.0, experts=16, top=4)
+# `--arch dosuvik`: the same widths, head counts, head sizes and vocabularies with Dosuvik layers in
+# the pattern window attention + dense, retention + experts, latent attention + experts, window
+# attention + experts: a window longer than the timed contexts, rotation on half of the head;
+# Digosun's key/value latents with a rotated key part of half a head; retention with the shape's
+# heads at the same widths; sixteen experts of a quarter of the dense feed-forward's width in four
+# groups of which two are kept, four per token.
+DOSUVIK = dict(window=8192, limit=7.0, experts=16, top=4, groups=(4, 2))
 CONTEXT = 2048          # cached tokens per request when decode is timed
 MAX_CONTEXT = 4096      # "benchmark at context 4096": positions the model is laid out for
 LONG_CONTEXT = 40960    # ... when the points at 8 k and 32 k cached tokens are measured too
@@ -303,14 +311,34 @@ def gikarax_config(shape: str, layers: int, positions: int) -> dict:
     return cfg
 
 
+def dosuvik_config(shape: str, layers: int, positions: int) -> dict:
+    q, z = SHAPES[shape], DOSUVIK
+    D, hd, H, G = q["hidden_size"], q["head_dim"], q["num_attention_heads"], q["num_key_value_heads"]
+    half = {"dims": hd // 2, "base": q["rope_theta"]}
+    window = dict(heads=H, kv_heads=G, dim=hd, vdim=hd, scale=hd ** -0.5, mask={"size": z["window"]}, rot=half)
+    latent = dict(heads=H, dim=hd, rot_dim=hd // 2, vdim=hd, kv_rank=DIGOSUN_SHAPES[shape]["kv_rank"],
+                  scale=(1.5 * hd) ** -0.5, rot=half)
+    retention = dict(heads=H, dim=hd, vdim=hd, rot={"dims": hd, "base": q["rope_theta"]},
+                     decay=[1.0 - 2.0 ** -(5.0 + 7.0 * h / max(1, H - 1)) for h in range(H)])
+    dense = {"kind": "dense", "ff": q["intermediate_size"], "limit": z["limit"]}
+    moe = {"kind": "moe", "expert": {"ff": q["intermediate_size"] // 4},
+           "router": {"experts": z["experts"], "top": z["top"],
+                      "groups": {"count": z["groups"][0], "keep": z["groups"][1]}}}
+    pattern = [("attention", window, dense), ("retention", retention, moe),
+               ("latent_attention", latent, moe), ("attention", window, moe)]
+    return {"architecture": "Dosuvik", "vocab": q["vocab_size"], "width": D,
+            "norm": {"eps": q["rms_norm_eps"]}, "max_positions": positions,
+            "layers": [dict(zip(("type", "mixer", "mlp"), pattern[i % 4])) for i in range(layers)]}
+
+
 ARCH = "qwen2"     # set by --arch; the other architectures build the same shapes with their layers
 
 
 def build_engine(shape: str, layers: int, max_tokens: int, max_requests: int, positions: int):
     import torch
 
-    from somi_inference_b200.config import (DapozenConfig, DigosunConfig, GikaraxConfig,
-                                            PoselornConfig, Qwen2Config)
+    from somi_inference_b200.config import (DapozenConfig, DigosunConfig, DosuvikConfig,
+                                            GikaraxConfig, PoselornConfig, Qwen2Config)
     from somi_inference_b200.engine import Engine
     from somi_inference_b200.parts import declared_tensors
     if ARCH == "digosun":
@@ -321,6 +349,8 @@ def build_engine(shape: str, layers: int, max_tokens: int, max_requests: int, po
         cfg = PoselornConfig.from_dict(poselorn_config(shape, layers, positions))
     elif ARCH == "gikarax":
         cfg = GikaraxConfig.from_dict(gikarax_config(shape, layers, positions))
+    elif ARCH == "dosuvik":
+        cfg = DosuvikConfig.from_dict(dosuvik_config(shape, layers, positions))
     else:
         cfg = Qwen2Config.from_dict(shape_config(shape, layers, positions))
     gen = torch.Generator(device="cuda").manual_seed(0)
@@ -520,7 +550,56 @@ def gikarax_sizes(cfg, batch: int) -> dict:
             "state_bytes_per_request": state, "window": min(windows)}
 
 
+def dosuvik_sizes(cfg, batch: int) -> dict:
+    """The same figures for a Dosuvik model.  A decode step of `batch` tokens reads at most
+    batch * top experts of a layer; a latent cache row holds kv_rank + rot_dim numbers, read once for
+    all heads; every matrix state is read and written once per request and step in float32 (5
+    flops per state entry and token)."""
+    D, V = cfg.width, cfg.vocab
+    params = read_params = small = kv = pair = state = 0
+    windows = [1 << 30]
+    for i, layer in enumerate(cfg.layers):
+        m = layer.mixer
+        if layer.type == "latent_attention":
+            inner = m["heads"] * m["vdim"]
+            p = (m["heads"] * (m["dim"] + m["rot_dim"]) + m["kv_rank"] + m["rot_dim"] + 2 * inner) * D \
+                + m["heads"] * (m["dim"] + m["vdim"]) * m["kv_rank"]
+            small += m["kv_rank"]
+            kv += 2 * (m["kv_rank"] + m["rot_dim"])
+            pair += 2 * m["heads"] * (2 * m["kv_rank"] + m["rot_dim"])
+        elif layer.type == "attention":
+            qk = (m["heads"] + m["kv_heads"]) * m["dim"]
+            p = (qk + m["kv_heads"] * m["vdim"] + m["heads"] * m["vdim"]) * D
+            small += qk + m["heads"]
+            kv += 2 * m["kv_heads"] * (m["dim"] + m["vdim"])
+            pair += 2 * m["heads"] * (m["dim"] + m["vdim"])
+            windows.append(m["mask"]["size"] if m.get("mask") else 1 << 30)
+        else:
+            p = (2 * m["heads"] * m["dim"] + 3 * m["heads"] * m["vdim"]) * D
+            p += 5 * m["heads"] * m["dim"] * m["vdim"] // 2
+            state += 2 * 4 * m["heads"] * m["dim"] * m["vdim"]
+        params += p
+        read_params += p
+        small += 2 * D
+        mlp = layer.mlp
+        if mlp is None:
+            continue
+        if mlp["kind"] == "dense":
+            params += 3 * D * mlp["ff"]
+            read_params += 3 * D * mlp["ff"]
+        else:
+            r = mlp["router"]
+            one = 3 * D * mlp["expert"]["ff"]
+            params += r["top"] * one + r["experts"] * D
+            read_params += min(r["experts"], batch * r["top"]) * one + r["experts"] * D
+    return {"weight_bytes": 2 * (read_params + small + V * D + D), "kv_bytes_per_token": kv,
+            "matmul_params": params, "head_params": V * D, "attn_flops_per_pair": pair,
+            "state_bytes_per_request": state, "window": min(windows)}
+
+
 def model_sizes(cfg, layers: int, batch: int = 1) -> dict:
+    if ARCH == "dosuvik":
+        return dosuvik_sizes(cfg, batch)
     if ARCH == "gikarax":
         return gikarax_sizes(cfg, batch)
     if ARCH == "digosun":
@@ -1120,12 +1199,15 @@ def main() -> int:
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", choices=["ours", "reference"], default="ours")
     ap.add_argument("--shape", choices=list(SHAPES), default="7b")
-    ap.add_argument("--arch", choices=["qwen2", "digosun", "dapozen", "poselorn", "gikarax"], default="qwen2",
+    ap.add_argument("--arch", choices=["qwen2", "digosun", "dapozen", "poselorn", "gikarax", "dosuvik"],
+                    default="qwen2",
                     help="with --only decode|prefill: the layer design the shape is built with "
                          "(digosun: latent attention under a window, gated branches; dapozen: "
                          "chunked attention with convolutions, Mamba-2 layers, table-routed experts; "
                          "gikarax: latent, capped window and causal attention, a gated linear "
-                         "attention, experts without gates, a loop)")
+                         "attention, experts without gates, a loop; dosuvik: window attention with "
+                         "turned values, retention, latent attention with a rotated key part, norms "
+                         "behind the branches, averages over depth)")
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the shape has")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--no-points", action="store_true",

@@ -44,7 +44,7 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ qkv, int row_stride,
                           const int* __restrict__ ctx_len, int nq, int nkv, int page_size,
                           float scale_log2e, int window, float cap_in, float cap_out,
                           const float* __restrict__ sinks, float* __restrict__ part_o,
-                          float* __restrict__ part_ml, int max_splits,
+                          float* __restrict__ part_ml, int max_splits, int merge_all,
                           __nv_bfloat16* __restrict__ out) {
     constexpr int CPR = HD / 8;
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -197,7 +197,7 @@ paged_decode_split_kernel(const __nv_bfloat16* __restrict__ qkv, int row_stride,
         }
     }
     __syncthreads();
-    const bool single = rg.n_splits - rg.first_split == 1;
+    const bool single = rg.n_splits - rg.first_split == 1 && !merge_all;
     for (int idx = tid; idx < G * HD; idx += kDecThreads) {
         const int g = idx / HD, d = idx - g * HD;
         float M = fmaxf(fmaxf(m_s[0][g], m_s[1][g]), fmaxf(m_s[2][g], m_s[3][g]));
@@ -225,7 +225,7 @@ int launch_decode(const void* qkv, int row_stride, int row_base, int req_base, i
                   const void* kcache, const void* vcache, const int* block_table, int bt_stride,
                   const int* ctx_len, int nq, int nkv, int page_size, float scale, int window,
                   float* part_o, float* part_ml, int max_splits, void* out, cudaStream_t stream,
-                  float softcap, const float* sinks) {
+                  float softcap, const float* sinks, const float* turn) {
     const size_t smem = static_cast<size_t>(kDecRows + 2 * kDecChunk) * HD * 2;
     if (smem > 48 * 1024)
         cudaFuncSetAttribute(paged_decode_split_kernel<HD>,
@@ -237,12 +237,12 @@ int launch_decode(const void* qkv, int row_stride, int row_base, int req_base, i
         block_table, bt_stride, ctx_len, nq, nkv, page_size, scale * 1.4426950408889634f, window,
         softcap > 0.f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.f,
         softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, sinks,
-        part_o, part_ml, max_splits, static_cast<__nv_bfloat16*>(out));
+        part_o, part_ml, max_splits, turn != nullptr ? 1 : 0, static_cast<__nv_bfloat16*>(out));
     int rc = launch_status();
-    if (rc != 0 || max_splits == 1) return rc;
+    if (rc != 0 || (max_splits == 1 && turn == nullptr)) return rc;
     return launch_decode_merge<HD>(part_o, part_ml, max_splits, kDecChunk, ctx_len, row_base, req_base,
                                    n_decode, nq, window, static_cast<__nv_bfloat16*>(out), stream,
-                                   sinks);
+                                   sinks, turn, turn != nullptr ? 1 : 0);
 }
 
 }  // namespace somi
@@ -260,12 +260,13 @@ SOMI_API int somi_decode_supported(int nq, int nkv, int hd) {
 
 // Scratch: part_o float32 [n_decode, nq, max_splits, hd], part_ml float32 [n_decode, nq, max_splits, 2].
 // `softcap` > 0: scores pass softcap * tanh(score / softcap); `sinks`: float32 [nq] scores that
-// join every softmax's denominator, or null.
+// join every softmax's denominator, or null; `turn`: float32 [rows of the step, hd / 2, 2] cosines and
+// sines by which the pairs of every head's output are turned back, or null.
 SOMI_API int somi_paged_attention_decode_shaped(
     const void* qkv, int row_stride, int row_base, int req_base, int n_decode, const void* kcache,
     const void* vcache, const int* block_table, int bt_stride, const int* ctx_len, int nq, int nkv,
     int hd, int page_size, float scale, int window, float softcap, const float* sinks,
-    float* part_o, float* part_ml, int max_splits, void* out, cudaStream_t stream) {
+    const float* turn, float* part_o, float* part_ml, int max_splits, void* out, cudaStream_t stream) {
     if (n_decode <= 0) return 0;
     if (!somi_decode_supported(nq, nkv, hd) || page_size <= 0 || max_splits <= 0 ||
         n_decode > 65535 || nkv > 65535)
@@ -273,7 +274,7 @@ SOMI_API int somi_paged_attention_decode_shaped(
 #define SOMI_DEC(HD)                                                                             \
     return launch_decode<HD>(qkv, row_stride, row_base, req_base, n_decode, kcache, vcache,      \
                              block_table, bt_stride, ctx_len, nq, nkv, page_size, scale, window, \
-                             part_o, part_ml, max_splits, out, stream, softcap, sinks)
+                             part_o, part_ml, max_splits, out, stream, softcap, sinks, turn)
     if (hd == 32) SOMI_DEC(32);
     if (hd == 64) SOMI_DEC(64);
     SOMI_DEC(128);
@@ -287,7 +288,7 @@ SOMI_API int somi_paged_attention_decode(
     void* out, cudaStream_t stream) {
     return somi_paged_attention_decode_shaped(qkv, row_stride, row_base, req_base, n_decode, kcache,
                                               vcache, block_table, bt_stride, ctx_len, nq, nkv, hd,
-                                              page_size, scale, window, 0.f, nullptr, part_o,
+                                              page_size, scale, window, 0.f, nullptr, nullptr, part_o,
                                               part_ml, max_splits, out, stream);
 }
 

@@ -52,7 +52,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map,
                         const int* __restrict__ block_table, int bt_stride,
                         const int* __restrict__ ctx_len, int nq, int nkv, int page_size,
                         float scale_log2e, int window, float* __restrict__ part_o,
-                        float* __restrict__ part_ml, int max_splits,
+                        float* __restrict__ part_ml, int max_splits, int merge_all,
                         __nv_bfloat16* __restrict__ out) {
     constexpr int CPR = HD / 8;
     constexpr int HALVES = HD / 64;
@@ -255,7 +255,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map,
     }
     const float L_lo = l_s[0][r_lo] + l_s[1][r_lo] + l_s[2][r_lo] + l_s[3][r_lo];
     const float L_hi = l_s[0][r_hi] + l_s[1][r_hi] + l_s[2][r_hi] + l_s[3][r_hi];
-    const bool single = rg.n_splits - rg.first_split == 1;
+    const bool single = rg.n_splits - rg.first_split == 1 && !merge_all;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
         const int g = half ? r_hi : r_lo;
@@ -307,7 +307,7 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
                          const int* __restrict__ block_table, int bt_stride,
                          const int* __restrict__ ctx_len, int nq, int nkv, int page_size,
                          float scale_log2e, int window, float* __restrict__ part_o,
-                         float* __restrict__ part_ml, int max_splits, int cpc,
+                         float* __restrict__ part_ml, int max_splits, int cpc, int merge_all,
                          __nv_bfloat16* __restrict__ out) {
     constexpr int CPR = HD / 8;
     constexpr int HALVES = HD / 64;
@@ -545,7 +545,7 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
     ring_compute_sync();
     const float L_lo = l_s[0][r_lo] + l_s[1][r_lo] + l_s[2][r_lo] + l_s[3][r_lo];
     const float L_hi = l_s[0][r_hi] + l_s[1][r_hi] + l_s[2][r_hi] + l_s[3][r_hi];
-    const bool single = rg.first_split / cpc == (rg.n_splits - 1) / cpc;
+    const bool single = rg.first_split / cpc == (rg.n_splits - 1) / cpc && !merge_all;
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
         const int g = half ? r_hi : r_lo;
@@ -575,7 +575,10 @@ int launch_tma_decode(const CUtensorMap* map, const void* qkv, int row_stride, i
                       int req_base, int n_decode, long long k_row0, long long v_row0,
                       const int* block_table, int bt_stride, const int* ctx_len, int nq, int nkv,
                       int page_size, float scale, int window, float* part_o, float* part_ml,
-                      int max_splits, void* out, cudaStream_t stream) {
+                      int max_splits, void* out, cudaStream_t stream, const float* sinks,
+                      const float* turn) {
+    // sinks and turned outputs are the merge kernel's: every request goes through it then
+    const int merge_all = sinks != nullptr || turn != nullptr;
     constexpr int TILE = (HD / 64) * kHalfBytes;
     const size_t smem = 2 * TILE + kTdRows * HD * 2 + kTdRows * kTdChunk * 2 + 1024;
     cudaFuncSetAttribute(paged_decode_tma_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -602,23 +605,24 @@ int launch_tma_decode(const CUtensorMap* map, const void* qkv, int row_stride, i
                    ring_smem, stream, *map, static_cast<const __nv_bfloat16*>(qkv), row_stride,
                    row_base, req_base, k_row0, v_row0, block_table, bt_stride, ctx_len, nq, nkv,
                    page_size, scale * 1.4426950408889634f, window, part_o, part_ml, max_splits, cpc,
-                   static_cast<__nv_bfloat16*>(out));
+                   merge_all, static_cast<__nv_bfloat16*>(out));
         int rc = launch_status();
-        if (rc != 0 || groups == 1) return rc;
+        if (rc != 0 || (groups == 1 && !merge_all)) return rc;
         return launch_decode_merge<HD>(part_o, part_ml, max_splits, kTdChunk * cpc, ctx_len, row_base,
                                        req_base, n_decode, nq, window,
-                                       static_cast<__nv_bfloat16*>(out), stream);
+                                       static_cast<__nv_bfloat16*>(out), stream, sinks, turn, merge_all);
     }
     dim3 grid(max_splits, nkv, n_decode);
     launch_pdl(paged_decode_tma_kernel<HD>, dim3(grid), dim3(kTdThreads), smem, stream, 
         *map, static_cast<const __nv_bfloat16*>(qkv), row_stride, row_base, req_base, k_row0,
         v_row0, block_table, bt_stride, ctx_len, nq, nkv, page_size,
-        scale * 1.4426950408889634f, window, part_o, part_ml, max_splits,
+        scale * 1.4426950408889634f, window, part_o, part_ml, max_splits, merge_all,
         static_cast<__nv_bfloat16*>(out));
     int rc = launch_status();
-    if (rc != 0 || max_splits == 1) return rc;
+    if (rc != 0 || (max_splits == 1 && !merge_all)) return rc;
     return launch_decode_merge<HD>(part_o, part_ml, max_splits, kTdChunk, ctx_len, row_base, req_base,
-                                   n_decode, nq, window, static_cast<__nv_bfloat16*>(out), stream);
+                                   n_decode, nq, window, static_cast<__nv_bfloat16*>(out), stream, sinks,
+                                   turn, merge_all);
 }
 
 }  // namespace somi
@@ -651,12 +655,15 @@ SOMI_API int somi_decode_tma_error() {
     return v;
 }
 
-// k_row0 / v_row0: first row, in the tensor map, of this run's key and value planes.
+// k_row0 / v_row0: first row, in the tensor map, of this run's key and value planes.  `sinks`: float32
+// [nq] scores that join every softmax's denominator, or null; `turn`: float32 [rows of the step, hd / 2, 2]
+// cosines and sines by which the pairs of every head's output are turned back, or null.
 SOMI_API int somi_paged_attention_decode_tma(
     const void* tensor_map, const void* qkv, int row_stride, int row_base, int req_base,
     int n_decode, long long k_row0, long long v_row0, const int* block_table, int bt_stride,
     const int* ctx_len, int nq, int nkv, int hd, int page_size, float scale, int window,
-    float* part_o, float* part_ml, int max_splits, void* out, cudaStream_t stream) {
+    const float* sinks, const float* turn, float* part_o, float* part_ml, int max_splits, void* out,
+    cudaStream_t stream) {
     if (n_decode <= 0) return 0;
     if (!somi_decode_tma_supported(nq, nkv, hd, page_size) || max_splits <= 0 ||
         n_decode > 65535 || nkv > 65535)
@@ -665,8 +672,8 @@ SOMI_API int somi_paged_attention_decode_tma(
     if (hd == 64)
         return launch_tma_decode<64>(map, qkv, row_stride, row_base, req_base, n_decode, k_row0,
                                      v_row0, block_table, bt_stride, ctx_len, nq, nkv, page_size,
-                                     scale, window, part_o, part_ml, max_splits, out, stream);
+                                     scale, window, part_o, part_ml, max_splits, out, stream, sinks, turn);
     return launch_tma_decode<128>(map, qkv, row_stride, row_base, req_base, n_decode, k_row0,
                                   v_row0, block_table, bt_stride, ctx_len, nq, nkv, page_size,
-                                  scale, window, part_o, part_ml, max_splits, out, stream);
+                                  scale, window, part_o, part_ml, max_splits, out, stream, sinks, turn);
 }

@@ -61,7 +61,8 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
                         long long v_row0, const int* __restrict__ block_table, int bt_stride,
                         const int* __restrict__ cu_q, const int* __restrict__ ctx_len,
                         const int* __restrict__ tiles, int nq, int nkv, int page_size,
-                        float scale_log2e, int window, __nv_bfloat16* __restrict__ out,
+                        float scale_log2e, int window, const float* __restrict__ sinks,
+                        const float2* __restrict__ turn, __nv_bfloat16* __restrict__ out,
                         int n_q_tiles) {
     constexpr int HALVES = HD / 64;
     constexpr int QTILE = HALVES * kPpQHalf;
@@ -390,23 +391,61 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
             ok = mbar_wait(smem_u32(&o_done[x]), 0, ok ? 400000 : 1) && ok;
             t5::fence_after();
             if (!ok) failed_s = 1;
+            // a sink: one more score in the denominator, without a value
+            if (sinks != nullptr) l += fast_exp2(sinks[head] * 1.4426950408889634f - m);
             const float inv = 1.0f / l;
             const int r = x * kPpBM + row;
             __nv_bfloat16* dst = out + static_cast<size_t>(row0 + r) * nq * HD + head * HD;
+            auto store8 = [](__nv_bfloat16* p, const float* y) {
+                uint4 w;
+                w.x = pack_bf16(y[0], y[1]);
+                w.y = pack_bf16(y[2], y[3]);
+                w.z = pack_bf16(y[4], y[5]);
+                w.w = pack_bf16(y[6], y[7]);
+                *reinterpret_cast<uint4*>(p) = w;
+            };
+            if (turn == nullptr) {
 #pragma unroll
-            for (int c = 0; c < HD / 32; ++c) {
-                uint32_t v[32];
-                t5::ld32_nowait(o_addr + c * 32, v);
-                t5::wait_ld();
-                if (r < rows) {
+                for (int c = 0; c < HD / 32; ++c) {
+                    uint32_t v[32];
+                    t5::ld32_nowait(o_addr + c * 32, v);
+                    t5::wait_ld();
+                    if (r < rows) {
 #pragma unroll
-                    for (int d = 0; d < 32; d += 8) {
-                        uint4 w;
-                        w.x = pack_bf16(__uint_as_float(v[d]) * inv, __uint_as_float(v[d + 1]) * inv);
-                        w.y = pack_bf16(__uint_as_float(v[d + 2]) * inv, __uint_as_float(v[d + 3]) * inv);
-                        w.z = pack_bf16(__uint_as_float(v[d + 4]) * inv, __uint_as_float(v[d + 5]) * inv);
-                        w.w = pack_bf16(__uint_as_float(v[d + 6]) * inv, __uint_as_float(v[d + 7]) * inv);
-                        *reinterpret_cast<uint4*>(dst + c * 32 + d) = w;
+                        for (int d = 0; d < 32; d += 8) {
+                            float y[8];
+#pragma unroll
+                            for (int j = 0; j < 8; ++j) y[j] = __uint_as_float(v[d + j]) * inv;
+                            store8(dst + c * 32 + d, y);
+                        }
+                    }
+                }
+            } else {
+                // the pairs (d, d + HD / 2) are turned back by the row's angles before they are rounded
+#pragma unroll
+                for (int c = 0; c < HD / 64; ++c) {
+                    uint32_t v[32], u[32];
+                    t5::ld32_nowait(o_addr + c * 32, v);
+                    t5::ld32_nowait(o_addr + HD / 2 + c * 32, u);
+                    t5::wait_ld();
+                    if (r < rows) {
+                        const float4* tr = reinterpret_cast<const float4*>(turn + static_cast<size_t>(row0 + r) * (HD / 2) + c * 32);
+#pragma unroll
+                        for (int d = 0; d < 32; d += 8) {
+                            float y0[8], y1[8];
+#pragma unroll
+                            for (int j = 0; j < 8; j += 2) {
+                                const float4 cs = tr[(d + j) / 2];          // two pairs' cosine, sine
+                                const float p0 = __uint_as_float(v[d + j]) * inv, q0 = __uint_as_float(u[d + j]) * inv;
+                                const float p1 = __uint_as_float(v[d + j + 1]) * inv, q1 = __uint_as_float(u[d + j + 1]) * inv;
+                                y0[j] = fmaf(p0, cs.x, q0 * cs.y);
+                                y1[j] = fmaf(q0, cs.x, -(p0 * cs.y));
+                                y0[j + 1] = fmaf(p1, cs.z, q1 * cs.w);
+                                y1[j + 1] = fmaf(q1, cs.z, -(p1 * cs.w));
+                            }
+                            store8(dst + c * 32 + d, y0);
+                            store8(dst + HD / 2 + c * 32 + d, y1);
+                        }
                     }
                 }
             }
@@ -426,7 +465,8 @@ template <int HD>
 int launch_prefill_pp(const CUtensorMap* q_map, const CUtensorMap* kv_map, long long k_row0,
                       long long v_row0, const int* block_table, int bt_stride, const int* cu_q,
                       const int* ctx_len, const int* tiles, int n_tiles, int nq, int nkv,
-                      int page_size, float scale, int window, void* out, cudaStream_t stream) {
+                      int page_size, float scale, int window, const float* sinks, const float* turn,
+                      void* out, cudaStream_t stream) {
     const size_t smem = 2 * (HD / 64) * kPpQHalf +
                         (pp_k_stages(HD) + pp_v_stages(HD)) * (HD / 64) * kPpKvHalf + 1024;
     cudaFuncSetAttribute(paged_prefill_pp_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -434,7 +474,8 @@ int launch_prefill_pp(const CUtensorMap* q_map, const CUtensorMap* kv_map, long 
     dim3 grid(static_cast<unsigned>(nq) * n_tiles);
     launch_pdl(paged_prefill_pp_kernel<HD>, grid, dim3(kPpThreads), smem, stream, *q_map, *kv_map,
                k_row0, v_row0, block_table, bt_stride, cu_q, ctx_len, tiles, nq, nkv, page_size,
-               scale * 1.4426950408889634f, window, static_cast<__nv_bfloat16*>(out), n_tiles);
+               scale * 1.4426950408889634f, window, sinks, reinterpret_cast<const float2*>(turn),
+               static_cast<__nv_bfloat16*>(out), n_tiles);
     return launch_status();
 }
 
@@ -458,19 +499,21 @@ SOMI_API int somi_prefill_pp_error() {
 }
 
 // `tiles`: int32 [n_tiles, 3] = (request, first row, rows <= 256) over the multi-token requests;
+// `sinks`, `turn`: as for the decode kernel (attention_decode_tma.cu), or null;
 // `q_map`: the projection buffer's map with boxes of 128 rows x 64 columns (as the one-tile kernel's).
 SOMI_API int somi_paged_attention_prefill_pp(
     const void* q_map, const void* kv_map, long long k_row0, long long v_row0,
     const int* block_table, int bt_stride, const int* cu_q, const int* ctx_len, const int* tiles,
-    int n_tiles, int nq, int nkv, int hd, int page_size, float scale, int window, void* out,
-    cudaStream_t stream) {
+    int n_tiles, int nq, int nkv, int hd, int page_size, float scale, int window, const float* sinks,
+    const float* turn, void* out, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     if (!somi_prefill_pp_supported(nq, nkv, hd, page_size)) return SOMI_ERR_UNSUPPORTED;
     const CUtensorMap* qm = static_cast<const CUtensorMap*>(q_map);
     const CUtensorMap* km = static_cast<const CUtensorMap*>(kv_map);
     if (hd == 64)
         return launch_prefill_pp<64>(qm, km, k_row0, v_row0, block_table, bt_stride, cu_q, ctx_len,
-                                     tiles, n_tiles, nq, nkv, page_size, scale, window, out, stream);
+                                     tiles, n_tiles, nq, nkv, page_size, scale, window, sinks, turn, out,
+                                     stream);
     return launch_prefill_pp<128>(qm, km, k_row0, v_row0, block_table, bt_stride, cu_q, ctx_len, tiles,
-                                  n_tiles, nq, nkv, page_size, scale, window, out, stream);
+                                  n_tiles, nq, nkv, page_size, scale, window, sinks, turn, out, stream);
 }

@@ -133,8 +133,8 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map,
                         const int* __restrict__ cu_q, const int* __restrict__ ctx_len,
                         const int* __restrict__ tiles, int nq, int nkv, int page_size,
                         float scale_log2e, int window, float cap_in, float cap_out,
-                        const float* __restrict__ sinks, __nv_bfloat16* __restrict__ out,
-                        int n_q_tiles) {
+                        const float* __restrict__ sinks, const float2* __restrict__ turn,
+                        __nv_bfloat16* __restrict__ out, int n_q_tiles) {
     constexpr int HALVES = HD / 64;
     constexpr int QTILE = HALVES * kFaHalf;              // bytes of the Q tile
     constexpr int TILE = HALVES * kFaKvHalf;             // bytes of a K or V tile
@@ -437,22 +437,51 @@ paged_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map,
                                ? fast_exp2(sinks[head] * 1.4426950408889634f - mm) : 0.f;
         const float inv = 1.0f / (w_me * l + w_ot * l_o + sink);
         const float a_me = w_me * inv, a_ot = w_ot * inv;
-        __nv_bfloat16* dst = out + static_cast<size_t>(row0 + row) * nq * HD + head * HD + half * (HD / 2);
+        __nv_bfloat16* dst = out + static_cast<size_t>(row0 + row) * nq * HD + head * HD;
+        // columns [col, col + 32) of the row: both key halves' accumulators, weighted
+        auto fetch = [&](int col, float (&v)[32]) {
+            float u[32];
+            fa_tmem_ld32(tmem_o + lane_addr + col, v);
+            fa_tmem_ld32(tmem_pv + (half ^ 1) * HD + lane_addr + col, u);
 #pragma unroll
-        for (int c = 0; c < HD / 64; ++c) {
-            float v[32], u[32];
-            fa_tmem_ld32(tmem_o + lane_addr + half * (HD / 2) + c * 32, v);
-            fa_tmem_ld32(tmem_pv + (half ^ 1) * HD + lane_addr + half * (HD / 2) + c * 32, u);
+            for (int d = 0; d < 32; ++d) v[d] = v[d] * a_me + u[d] * a_ot;
+        };
+        auto store32 = [](__nv_bfloat16* p, const float (&v)[32]) {
+#pragma unroll
+            for (int d = 0; d < 32; d += 8) {
+                uint4 w;
+                w.x = pack_bf16(v[d], v[d + 1]);
+                w.y = pack_bf16(v[d + 2], v[d + 3]);
+                w.z = pack_bf16(v[d + 4], v[d + 5]);
+                w.w = pack_bf16(v[d + 6], v[d + 7]);
+                *reinterpret_cast<uint4*>(p + d) = w;
+            }
+        };
+        if (turn == nullptr) {
+#pragma unroll
+            for (int c = 0; c < HD / 64; ++c) {
+                float v[32];
+                fetch(half * (HD / 2) + c * 32, v);
+                if (row < rows) store32(dst + half * (HD / 2) + c * 32, v);
+            }
+        } else if (HD == 128 || half == 0) {
+            // the pairs (d, d + HD / 2) are turned back by the row's angles before they are rounded: a
+            // thread takes 32 pairs (heads of 64 have no more, which are the first half's threads')
+            const int col = HD == 128 ? half * 32 : 0;
+            float p[32], q[32];
+            fetch(col, p);
+            fetch(col + HD / 2, q);
             if (row < rows) {
+                const float2* tr = turn + static_cast<size_t>(row0 + row) * (HD / 2) + col;
 #pragma unroll
-                for (int d = 0; d < 32; d += 8) {
-                    uint4 w;
-                    w.x = pack_bf16(v[d] * a_me + u[d] * a_ot, v[d + 1] * a_me + u[d + 1] * a_ot);
-                    w.y = pack_bf16(v[d + 2] * a_me + u[d + 2] * a_ot, v[d + 3] * a_me + u[d + 3] * a_ot);
-                    w.z = pack_bf16(v[d + 4] * a_me + u[d + 4] * a_ot, v[d + 5] * a_me + u[d + 5] * a_ot);
-                    w.w = pack_bf16(v[d + 6] * a_me + u[d + 6] * a_ot, v[d + 7] * a_me + u[d + 7] * a_ot);
-                    *reinterpret_cast<uint4*>(dst + c * 32 + d) = w;
+                for (int d = 0; d < 32; ++d) {
+                    const float2 cs = tr[d];
+                    const float a = p[d], b = q[d];
+                    p[d] = fmaf(a, cs.x, b * cs.y);
+                    q[d] = fmaf(b, cs.x, -(a * cs.y));
                 }
+                store32(dst + col, p);
+                store32(dst + col + HD / 2, q);
             }
         }
     }
@@ -471,7 +500,7 @@ int launch_prefill_tc(const CUtensorMap* q_map, const CUtensorMap* kv_map, long 
                       long long v_row0, const int* block_table, int bt_stride, const int* cu_q,
                       const int* ctx_len, const int* tiles, int n_tiles, int nq, int nkv,
                       int page_size, float scale, int window, float softcap, const float* sinks,
-                      void* out, cudaStream_t stream) {
+                      const float* turn, void* out, cudaStream_t stream) {
     const size_t smem = (HD / 64) * kFaHalf + 2 * fa_stages(HD) * (HD / 64) * kFaKvHalf + 4 * kFaHalf + 1024;
     cudaFuncSetAttribute(paged_prefill_tc_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                          (int)smem);
@@ -481,7 +510,7 @@ int launch_prefill_tc(const CUtensorMap* q_map, const CUtensorMap* kv_map, long 
                scale * 1.4426950408889634f, window,
                softcap > 0.f ? 2.0f * 1.4426950408889634f * scale / softcap : 0.f,
                softcap > 0.f ? softcap * 1.4426950408889634f : 0.f, sinks,
-               static_cast<__nv_bfloat16*>(out), n_tiles);
+               reinterpret_cast<const float2*>(turn), static_cast<__nv_bfloat16*>(out), n_tiles);
     return launch_status();
 }
 
@@ -516,12 +545,12 @@ SOMI_API int somi_make_q_tensor_map(void* map_out, const void* qkv, long long to
 
 // `tiles`: int32 [n_tiles, 3] = (request, first row, rows <= 128) over the multi-token requests.
 // `softcap` > 0: scores pass softcap * tanh(score / softcap); `sinks`: float32 [nq] scores that
-// join every softmax's denominator, or null.
+// join every softmax's denominator, or null; `turn`: as for the decode kernel (attention_decode_tma.cu).
 SOMI_API int somi_paged_attention_prefill_tc_shaped(
     const void* q_map, const void* kv_map, long long k_row0, long long v_row0,
     const int* block_table, int bt_stride, const int* cu_q, const int* ctx_len, const int* tiles,
     int n_tiles, int nq, int nkv, int hd, int page_size, float scale, int window, float softcap,
-    const float* sinks, void* out, cudaStream_t stream) {
+    const float* sinks, const float* turn, void* out, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     if (!somi_prefill_tc_supported(nq, nkv, hd, page_size) ) return SOMI_ERR_UNSUPPORTED;
     const CUtensorMap* qm = static_cast<const CUtensorMap*>(q_map);
@@ -529,10 +558,10 @@ SOMI_API int somi_paged_attention_prefill_tc_shaped(
     if (hd == 64)
         return launch_prefill_tc<64>(qm, km, k_row0, v_row0, block_table, bt_stride, cu_q, ctx_len,
                                      tiles, n_tiles, nq, nkv, page_size, scale, window, softcap,
-                                     sinks, out, stream);
+                                     sinks, turn, out, stream);
     return launch_prefill_tc<128>(qm, km, k_row0, v_row0, block_table, bt_stride, cu_q, ctx_len, tiles,
-                                  n_tiles, nq, nkv, page_size, scale, window, softcap, sinks, out,
-                                  stream);
+                                  n_tiles, nq, nkv, page_size, scale, window, softcap, sinks, turn,
+                                  out, stream);
 }
 
 SOMI_API int somi_paged_attention_prefill_tc(
@@ -542,6 +571,6 @@ SOMI_API int somi_paged_attention_prefill_tc(
     cudaStream_t stream) {
     return somi_paged_attention_prefill_tc_shaped(q_map, kv_map, k_row0, v_row0, block_table,
                                                   bt_stride, cu_q, ctx_len, tiles, n_tiles, nq, nkv,
-                                                  hd, page_size, scale, window, 0.f, nullptr, out,
+                                                  hd, page_size, scale, window, 0.f, nullptr, nullptr, out,
                                                   stream);
 }

@@ -23,7 +23,7 @@ namespace somi {
 // if write_back: x_out[row] = x.  out[b] = x in TO, or with `weight` x / sqrt(mean(x^2) + eps) * weight;
 // row = rows ? rows[b] : b.  V vectors of four columns a thread, kept in registers.
 template <typename TD, typename TO, int V>
-__global__ void __launch_bounds__(1024)
+__global__ void __launch_bounds__(V == 4 ? 512 : 1024)
 stream_update_kernel(const float* x_in, float* x_out,       // (may be the same rows)
                      const TD* __restrict__ delta, int splits, long long split_stride,
                      const void* __restrict__ weight_b, int wb_dtype, float eps_b,
@@ -476,14 +476,14 @@ SOMI_API int somi_stream_update(const float* x_in, float* x_out, const void* del
     if (H <= 0 || (splits > 1 && delta_dtype != SOMI_F32) ||
         (coef != nullptr && (n < 1 || start == nullptr || results == nullptr)))
         return SOMI_ERR_UNSUPPORTED;
-    const bool vec4 = (H & 3) == 0 && H <= 16384 && aligned16(x_in) && aligned16(x_out) && aligned16(delta) &&
+    const bool vec4 = (H & 3) == 0 && H <= 8192 && aligned16(x_in) && aligned16(x_out) && aligned16(delta) &&
                       aligned16(weight_b) && aligned16(start) && aligned16(results) && aligned16(weight) &&
                       aligned16(out) && (split_stride & 3) == 0 && (result_stride & 3) == 0;
     // few rows (a decode step): a thread per four columns, every load of the row in flight at once
     const int vecs = (H + 3) / 4;
     int v = n_out <= 512 ? 1 : 4;
     if (vecs < 64 * v) v = 1;
-    while (v < 4 && (vecs + v - 1) / v > 1024) v *= 2;
+    if (v == 1 && vecs > 1024) v = 2;                     // (a CTA of V = 4 has at most 512 threads)
     const int threads = max(32, (((vecs + v - 1) / v + 31) / 32) * 32);
 #define SOMI_SU_ARGS(TD, TO)                                                                       \
     x_in, x_out, static_cast<const TD*>(delta), splits, split_stride, weight_b, wb_dtype, eps_b,   \

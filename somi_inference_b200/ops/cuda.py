@@ -291,7 +291,7 @@ class CudaOps:
 
     def paged_attention(self, qkv, kcache, vcache, batch, group, nq, nkv, hd, scale, window,
                         out, storage=None, value_dim=None, chunk=None, gate=None,
-                        gate_per_head=False, softcap=None, sinks=None) -> None:
+                        gate_per_head=False, softcap=None, sinks=None, turn=None) -> None:
         """Attention of every token of the step over the cache (keys/values already stored).
 
         In bfloat16 with head sizes 32/64/128, portions of prompts go to the tensor-core
@@ -302,10 +302,12 @@ class CudaOps:
         value width] (rows may lie further apart); the output is multiplied by their sigmoid;
         with `gate_per_head` the logits are [T, nq], one per token and head.  `softcap`: scores
         pass cap * tanh(score / cap); `sinks`: float32 [nq] scores that join the softmax's
-        denominator without a key.  With capped scores or sinks, bfloat16 prompt portions of head
-        sizes 64/128 run the one-tile tcgen05 kernel (or the `mma.sync` kernel that TMA feeds) and
-        single tokens the cp.async split-KV kernel; a per-head gate is then a kernel of its own
-        behind them.
+        denominator without a key; `turn`: float32 [T, value width / 2, 2] cosines and sines by which
+        the pairs (m, m + half) of every head's output are turned back.  bfloat16 head sizes 64/128:
+        every tcgen05 prompt kernel and every split-KV kernel takes sinks and turns (the merge does,
+        for single tokens); capped scores run the one-tile tcgen05 kernel (or the `mma.sync` kernel
+        that TMA feeds) and the cp.async split-KV kernel.  A gate, and a turn behind the other
+        kernels, is a kernel of its own behind them.
         """
         _check(qkv, kcache, vcache, out, group.block_table)
         assert kcache.dtype == qkv.dtype
@@ -322,6 +324,12 @@ class CudaOps:
         if sinks is not None:
             _check(sinks)
             assert sinks.dtype == torch.float32 and sinks.numel() == nq
+        if turn is not None:
+            _check(turn)
+            assert turn.dtype == torch.float32 and tuple(turn.shape) == (out.shape[0], vd // 2, 2)
+            if gate is not None or vd % 2:
+                raise KernelError("turned outputs come in pairs and without a gate")
+        prefill_turned = decode_turned = False      # whether the rows' kernel turned them
         n_decode = batch.num_requests - batch.num_prefill_requests
         # what the tensor-core kernels compute; they fetch query rows in 16-byte pieces
         plain = vd == hd and qkv.shape[1] % 8 == 0
@@ -333,7 +341,8 @@ class CudaOps:
                                and self.prefill_supported(nq, nkv, hd, qkv.dtype))
         shaped_tc = False
         if shaped and tensor_core_prefill:
-            # two kernels shape scores: the one-tile tcgen05 kernel and the TMA-fed mma.sync one
+            # capped scores: the one-tile tcgen05 kernel and the TMA-fed mma.sync one; sinks: these and
+            # the two-tile kernel
             geometry = (ctypes.c_int(nq), ctypes.c_int(nkv), ctypes.c_int(hd), ctypes.c_int(page_size))
             shaped_tc = (self.use_tc_prefill and storage is not None
                          and bool(self.lib.somi_prefill_tc_supported(*geometry)))
@@ -353,7 +362,12 @@ class CudaOps:
             row_bytes = hd * 2
             # (the two-tile kernel has half as many CTAs: below one per SM the one-tile kernel,
             # with twice as many, is the faster: 0.5B shape at 2,048 tokens 123 vs 148 TFLOP/s)
-            if shaped_tc:
+            two_tiles = (cap == 0.0 and self.use_pp_prefill and storage is not None and qkv.shape[1] % 8 == 0
+                         and batch.tiles[self.prefill_pp_q_tile].shape[0] * nq >= self.pp_prefill_min_ctas
+                         and bool(self.lib.somi_prefill_pp_supported(*sizes)))
+            if (shaped_tc or (turn is not None and self.use_tc_prefill and storage is not None
+                              and bool(self.lib.somi_prefill_tc_supported(*sizes)))) and not two_tiles:
+                prefill_turned = True
                 tiles = batch.tiles[self.prefill_tc_q_tile]
                 rc = self.lib.somi_paged_attention_prefill_tc_shaped(
                     ctypes.c_void_p(self._q_tensor_map(qkv)),
@@ -363,10 +377,10 @@ class CudaOps:
                     _ptr(group.block_table), ctypes.c_int(group.width), _ptr(batch.cu_q),
                     _ptr(batch.ctx_len), _ptr(tiles), ctypes.c_int(tiles.shape[0]), *sizes,
                     ctypes.c_float(scale), ctypes.c_int(win), ctypes.c_float(cap), _ptr(sinks),
-                    _ptr(out), self._stream())
+                    _ptr(turn), _ptr(out), self._stream())
                 self._done(rc, "paged_attention_prefill_tc")
                 kernel = "attention_prefill_tcgen05"
-            elif shaped:
+            elif shaped and not two_tiles:
                 tiles = batch.tiles[self.prefill_q_tile]
                 rc = self.lib.somi_paged_attention_prefill_tma_shaped(
                     ctypes.c_void_p(self._kv_tensor_map(storage, hd, page_size)), _ptr(qkv),
@@ -379,9 +393,8 @@ class CudaOps:
                     _ptr(out), self._stream())
                 self._done(rc, "paged_attention_prefill_tma")
                 kernel = "attention_prefill_tma"
-            elif (self.use_pp_prefill and storage is not None and qkv.shape[1] % 8 == 0
-                    and batch.tiles[self.prefill_pp_q_tile].shape[0] * nq >= self.pp_prefill_min_ctas
-                    and bool(self.lib.somi_prefill_pp_supported(*sizes))):
+            elif two_tiles:
+                prefill_turned = True
                 tiles = batch.tiles[self.prefill_pp_q_tile]
                 rc = self.lib.somi_paged_attention_prefill_pp(
                     ctypes.c_void_p(self._q_tensor_map(qkv)),
@@ -390,7 +403,8 @@ class CudaOps:
                     ctypes.c_longlong((vcache.data_ptr() - storage.data_ptr()) // row_bytes),
                     _ptr(group.block_table), ctypes.c_int(group.width), _ptr(batch.cu_q),
                     _ptr(batch.ctx_len), _ptr(tiles), ctypes.c_int(tiles.shape[0]), *sizes,
-                    ctypes.c_float(scale), ctypes.c_int(win), _ptr(out), self._stream())
+                    ctypes.c_float(scale), ctypes.c_int(win), _ptr(sinks), _ptr(turn), _ptr(out),
+                    self._stream())
                 self._done(rc, "paged_attention_prefill_pp")
                 kernel = "attention_prefill_tcgen05_pingpong"
             elif (self.use_tc_prefill and storage is not None and qkv.shape[1] % 8 == 0
@@ -457,7 +471,8 @@ class CudaOps:
             max_splits = -(-group.width * page_size // chunk)
             n_o = n_decode * nq * max_splits * hd
             ws = self._scratch(n_o + n_decode * nq * max_splits * 2, qkv.device)
-            tma = (not shaped and self.use_tma_decode and storage is not None and bool(
+            decode_turned = True
+            tma = (cap == 0.0 and self.use_tma_decode and storage is not None and bool(
                 self.lib.somi_decode_tma_supported(ctypes.c_int(nq), ctypes.c_int(nkv),
                                                    ctypes.c_int(hd), ctypes.c_int(page_size))))
             if tma:
@@ -471,8 +486,8 @@ class CudaOps:
                     ctypes.c_longlong(k_row0), ctypes.c_longlong(v_row0),
                     _ptr(group.block_table), ctypes.c_int(group.width), _ptr(batch.ctx_len),
                     ctypes.c_int(nq), ctypes.c_int(nkv), ctypes.c_int(hd),
-                    ctypes.c_int(page_size), ctypes.c_float(scale), ctypes.c_int(win),
-                    ctypes.c_void_p(ws.data_ptr()), ctypes.c_void_p(ws.data_ptr() + 4 * n_o),
+                    ctypes.c_int(page_size), ctypes.c_float(scale), ctypes.c_int(win), _ptr(sinks),
+                    _ptr(turn), ctypes.c_void_p(ws.data_ptr()), ctypes.c_void_p(ws.data_ptr() + 4 * n_o),
                     ctypes.c_int(max_splits), _ptr(out), self._stream())
             else:
                 rc = self.lib.somi_paged_attention_decode_shaped(
@@ -481,12 +496,12 @@ class CudaOps:
                     _ptr(kcache), _ptr(vcache), _ptr(group.block_table),
                     ctypes.c_int(group.width), _ptr(batch.ctx_len), ctypes.c_int(nq),
                     ctypes.c_int(nkv), ctypes.c_int(hd), ctypes.c_int(page_size),
-                    ctypes.c_float(scale), ctypes.c_int(win), ctypes.c_float(cap), _ptr(sinks),
+                    ctypes.c_float(scale), ctypes.c_int(win), ctypes.c_float(cap), _ptr(sinks), _ptr(turn),
                     ctypes.c_void_p(ws.data_ptr()),
                     ctypes.c_void_p(ws.data_ptr() + 4 * n_o), ctypes.c_int(max_splits),
                     _ptr(out), self._stream())
             self._done(rc, "paged_attention_decode")
-            if max_splits > 1:
+            if max_splits > 1 or turn is not None or (tma and sinks is not None):
                 self.launches += 1
             if trace.active():
                 trace.note("attention_decode_tma" if tma else "attention_decode_cp_async",
@@ -495,6 +510,11 @@ class CudaOps:
                                                  qkv.element_size(), win),
                            detail="with merge" if max_splits > 1 else "")
 
+        if turn is not None:
+            first = batch.num_prefill_tokens if prefill_turned else 0
+            last = batch.num_prefill_tokens if decode_turned else batch.num_tokens
+            if first < last:
+                self.turn_back(out[first:last], turn[first:last], nq, vd)
         if gate is not None and (tensor_core_prefill or split):
             # the generic kernel applied the gate to its own rows only
             first = 0 if tensor_core_prefill else batch.num_prefill_tokens

@@ -164,8 +164,6 @@ class NormedAttentionMixer:
                             self.key_dim, self.scale, self.window, out, storage=paged.storage,
                             value_dim=self.value_dim,
                             gate=qkv[:, self.gate_at:self.gate_at + self.heads] if self.head_gate else None,
-                            gate_per_head=self.head_gate, softcap=self.softcap, sinks=self.sinks)
-        if turn is not None:
-            ops.turn_back(out, turn, self.heads, self.value_dim)
+                            gate_per_head=self.head_gate, softcap=self.softcap, sinks=self.sinks, turn=turn)
         partial = self.out.partial_sums(out)
         return partial if partial is not None else self.out(out)
