@@ -413,14 +413,24 @@ __global__ void turn_back_kernel(T* __restrict__ x, const float2* __restrict__ t
 // elements behind it.  Written: cache row of the token [rank + rot] = (latent / rms * weight | turned
 // key part), and into qa [H, T, rank + rot] the turned tail of every query behind column `rank`
 // (the columns before it are another kernel's).  Pairs: i and i + rot / 2, or neighbours.
-// One CTA per token; sines and cosines are formed once per token.
+// One CTA per token; sines and cosines are formed once per token.  `vec2`: two neighbours at once
+// (neighbouring pairs, every offset even).
+__device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 load2(const __nv_bfloat16* p) {
+    return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+}
+__device__ __forceinline__ void store2(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+__device__ __forceinline__ void store2(__nv_bfloat16* p, float a, float b) {
+    *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_rotary_store_kernel(const T* __restrict__ x, long long stride, int q_at, int H, int qd, int rot,
                            int c_at, int rank, int neighbours, const int* __restrict__ positions,
                            const double* __restrict__ inv_freq, const void* __restrict__ weight,
                            int w_dtype, float eps, const int* __restrict__ slot_map, T* __restrict__ cache,
-                           T* __restrict__ qa, int n_tokens) {
+                           T* __restrict__ qa, int n_tokens, int vec2) {
     extern __shared__ float2 cs_s[];                       // [rot / 2]
     __shared__ float scratch[33];
     pdl_launch_dependents();
@@ -431,17 +441,32 @@ latent_rotary_store_kernel(const T* __restrict__ x, long long stride, int q_at, 
     const double pos = static_cast<double>(positions[t]);
     for (int i = tid; i < half; i += nthr) cs_s[i] = turn_by(pos, inv_freq[i]);
     float ss = 0.f;
-    for (int e = tid; e < rank; e += nthr) {
-        const float f = to_float(row[c_at + e]);
-        ss = fmaf(f, f, ss);
+    if (vec2) {
+        for (int e = 2 * tid; e < rank; e += 2 * nthr) {
+            const float2 f = load2(row + c_at + e);
+            ss = fmaf(f.x, f.x, fmaf(f.y, f.y, ss));
+        }
+    } else {
+        for (int e = tid; e < rank; e += nthr) {
+            const float f = to_float(row[c_at + e]);
+            ss = fmaf(f, f, ss);
+        }
     }
     ss = block_sum(ss, scratch);
     __syncthreads();
     const float inv = 1.0f / sqrtf(ss / static_cast<float>(rank) + eps);
     if (slot_map != nullptr) {
         T* dst = cache + static_cast<size_t>(slot_map[t]) * W;
-        for (int e = tid; e < rank; e += nthr)
-            dst[e] = from_float<T>(to_float(row[c_at + e]) * inv * load_as_float(weight, w_dtype, e));
+        if (vec2) {
+            for (int e = 2 * tid; e < rank; e += 2 * nthr) {
+                const float2 f = load2(row + c_at + e);
+                store2(dst + e, f.x * inv * load_as_float(weight, w_dtype, e),
+                       f.y * inv * load_as_float(weight, w_dtype, e + 1));
+            }
+        } else {
+            for (int e = tid; e < rank; e += nthr)
+                dst[e] = from_float<T>(to_float(row[c_at + e]) * inv * load_as_float(weight, w_dtype, e));
+        }
     }
     for (int it = tid; it < (H + 1) * half; it += nthr) {
         const int h = it / half, j = it - h * half;
@@ -452,6 +477,11 @@ latent_rotary_store_kernel(const T* __restrict__ x, long long stride, int q_at, 
         else if (slot_map != nullptr) dst = cache + static_cast<size_t>(slot_map[t]) * W + rank;
         else continue;
         const float2 cs = cs_s[j];
+        if (vec2) {
+            const float2 f = load2(src + e0);
+            store2(dst + e0, fmaf(f.x, cs.x, -(f.y * cs.y)), fmaf(f.y, cs.x, f.x * cs.y));
+            continue;
+        }
         const float u = to_float(src[e0]), v = to_float(src[e1]);
         dst[e0] = from_float<T>(fmaf(u, cs.x, -(v * cs.y)));
         dst[e1] = from_float<T>(fmaf(v, cs.x, u * cs.y));
@@ -570,11 +600,13 @@ SOMI_API int somi_latent_rotary_store(const void* x, int dtype, long long stride
     if (T <= 0) return 0;
     if (H <= 0 || qd < 0 || rot < 0 || (rot & 1) || rot > 4096 || rank <= 0) return SOMI_ERR_UNSUPPORTED;
     const size_t smem = sizeof(float2) * (rot / 2 + 1);
+    const int vec2 = neighbours && ((q_at | qd | c_at | rank) & 1) == 0 && (stride & 1) == 0 && aligned16(x) &&
+                     aligned16(cache) && aligned16(qa);
 #define SOMI_LAUNCH_LRS(TT)                                                                        \
     launch_pdl(latent_rotary_store_kernel<TT>, dim3(T), dim3(256), smem, stream,                   \
                static_cast<const TT*>(x), stride, q_at, H, qd, rot, c_at, rank, neighbours,        \
                positions, inv_freq, weight, w_dtype, eps, slot_map, static_cast<TT*>(cache),       \
-               static_cast<TT*>(qa), T)
+               static_cast<TT*>(qa), T, vec2)
     if (dtype == SOMI_F32) SOMI_LAUNCH_LRS(float);
     else SOMI_LAUNCH_LRS(__nv_bfloat16);
 #undef SOMI_LAUNCH_LRS
