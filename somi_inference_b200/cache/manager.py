@@ -9,7 +9,7 @@ block list and token count, two-phase use (`allocate_slots` before the forward,
 What this manager does differently:
 
 * Runs of the schedule are put into *groups* by what they need (kv heads, key
-  width, value width, window).  Each group has its own page pool, its own device
+  width, value width, window, kept first positions).  Each group has its own page pool, its own device
   storage and its own block table per request.  Where keys and values have the
   same width the storage is one tensor `[runs_in_group, 2, num_pages, kv_heads,
   page_size, head_dim]` (a page of one kv head is contiguous, and one tensor map
@@ -17,7 +17,8 @@ What this manager does differently:
   `[runs_in_group, num_pages, kv_heads, page_size, width]`.  Runs that attend over all keys and runs that only
   ever read a window therefore never compete for, or waste, each other's pages.
 * A window group gives pages back as soon as every position in them has fallen
-  out of the window (`commit`); the block table keeps -1 in their place.
+  out of the window (`commit`); the block table keeps -1 in their place.  Where first
+  positions stay readable beside the window, their pages are held to the end.
 * A run that reads another run's cache shares that run's pages and block tables; state of
   fixed size is never shared: every run has the tensors its own layer asked for.
 * Every request also gets a *state slot*: an index into per-run tensors of fixed
@@ -88,12 +89,20 @@ class _Group:
                                        needs.value_width), dtype=dtype, device=device)
         # host block tables, one row per state slot (= per live request)
         self.tables = np.full((max_requests, max_blocks), FREED, dtype=np.int32)
-        self.first_live = np.zeros(max_requests, dtype=np.int64)  # first block not yet given back
+        # blocks of first positions that stay readable, whatever falls out of the window
+        self.kept = -(-needs.keep_first // page_size) if needs.window is not None else 0
+        self.first_live = np.zeros(max_requests, dtype=np.int64)  # behind those: first block not yet given back
         self.num_blocks = np.zeros(max_requests, dtype=np.int64)  # blocks ever taken
 
     def blocks_needed(self, slot: int, new_len: int) -> int:
         want = -(-new_len // self.page_size)
         return max(0, want - int(self.num_blocks[slot]))
+
+    def held(self, slot: int) -> list[int]:
+        """The pages a request holds, in the order of their positions."""
+        first, last = int(self.first_live[slot]), int(self.num_blocks[slot])
+        row = self.tables[slot]
+        return [int(p) for p in row[:min(self.kept, first, last)]] + [int(p) for p in row[first:last]]
 
 
 class CacheManager:
@@ -120,8 +129,8 @@ class CacheManager:
         for run, (needs, owner) in enumerate(zip(needs_per_run, owner_of_run)):
             if owner is None and needs is not None and needs.paged is not None:
                 p = needs.paged
-                by_key.setdefault((p.num_kv_heads, p.head_dim, p.window, p.value_width),
-                                  []).append(run)
+                by_key.setdefault((p.num_kv_heads, p.head_dim, p.window, p.value_width,
+                                   p.keep_first if p.window is not None else 0), []).append(run)
         for key, runs in by_key.items():
             needs = PagedKVNeeds(*key)
             self.groups.append(_Group(needs, runs, num_pages, page_size, max_requests,
@@ -246,7 +255,7 @@ class CacheManager:
                 continue
             # the next query sits at position `length` and reads keys > length - window
             first_needed = max(0, self._len[req] - g.needs.window + 1) // self.page_size
-            first = int(g.first_live[slot])
+            first = max(int(g.first_live[slot]), g.kept)
             if first_needed > first:
                 g.pool.give_back([int(p) for p in g.tables[slot, first:first_needed]])
                 g.tables[slot, first:first_needed] = FREED
@@ -258,9 +267,8 @@ class CacheManager:
         del self._len[req]
         del self._reserved[req]
         for g in self.groups:
-            first, last = int(g.first_live[slot]), int(g.num_blocks[slot])
-            g.pool.give_back([int(p) for p in g.tables[slot, first:last]])
-            g.tables[slot, :last] = FREED
+            g.pool.give_back(g.held(slot))
+            g.tables[slot, :int(g.num_blocks[slot])] = FREED
             g.first_live[slot] = 0
             g.num_blocks[slot] = 0
         self._slots.give_back([slot])
@@ -274,9 +282,7 @@ class CacheManager:
         return int(self.groups[group].num_blocks[slot])
 
     def held_pages(self, req: object, group: int) -> list[int]:
-        slot = self._slot_of[req]
-        g = self.groups[group]
-        return [int(p) for p in g.tables[slot, int(g.first_live[slot]):int(g.num_blocks[slot])]]
+        return self.groups[group].held(self._slot_of[req])
 
     def check_consistency(self) -> None:
         """Every page is either free or held by exactly one live request (used by tests)."""

@@ -1,5 +1,7 @@
 """Configuration: typed architecture configs, the model spec they produce, the registry."""
 
+from .bibalix import ARCHITECTURE as BIBALIX_ARCHITECTURE
+from .bibalix import BibalixConfig
 from .dapozen import ARCHITECTURE as DAPOZEN_ARCHITECTURE
 from .dapozen import DapozenConfig
 from .digosun import ARCHITECTURE as DIGOSUN_ARCHITECTURE
@@ -22,10 +24,11 @@ register_architecture(DAPOZEN_ARCHITECTURE, DapozenConfig)
 register_architecture(POSELORN_ARCHITECTURE, PoselornConfig)
 register_architecture(GIKARAX_ARCHITECTURE, GikaraxConfig)
 register_architecture(DOSUVIK_ARCHITECTURE, DosuvikConfig)
+register_architecture(BIBALIX_ARCHITECTURE, BibalixConfig)
 
 __all__ = ["ConfigError", "Qwen2Config", "QWEN2_ARCHITECTURE", "DigosunConfig",
            "DIGOSUN_ARCHITECTURE", "DapozenConfig", "DAPOZEN_ARCHITECTURE", "PoselornConfig",
            "POSELORN_ARCHITECTURE", "GikaraxConfig", "GIKARAX_ARCHITECTURE", "DosuvikConfig",
-           "DOSUVIK_ARCHITECTURE", "LayerSpec", "ModelSpec", "PartSpec", "RunSpec",
+           "DOSUVIK_ARCHITECTURE", "BibalixConfig", "BIBALIX_ARCHITECTURE", "LayerSpec", "ModelSpec", "PartSpec", "RunSpec",
            "config_class_for", "load_config", "register_architecture", "supported_architectures",
            "unregister_architecture"]

@@ -11,11 +11,19 @@
 // page_size consecutive rows.
 //
 // Needs head_dim 64 or 128 and a page size that is a multiple of 8 and divides 128.
+//
+// `maps` = 2: a key row of head_dim elements holds two keys of half that width over one value
+// (attention in two maps, see two_maps.cuh).  Every head of the group is then two MMA rows, its
+// query's first half with zeros behind it and its second half with zeros in front, so the
+// scores of both maps come from one product over the same key tile; the merge takes the
+// difference of the maps.  `keep`: keys below that position stay visible beside a window; the
+// chunks in between are skipped (TdRange numbers the chunks that are left).
 #include <algorithm>
 
 #include "attention_merge.cuh"
 #include "mma.cuh"
 #include "tma.cuh"
+#include "two_maps.cuh"
 
 namespace somi {
 
@@ -32,15 +40,30 @@ __device__ __forceinline__ int tma_tile_offset(int key, int chunk) {
     return (chunk >> 3) * kHalfBytes + key * 128 + (((chunk & 7) ^ (key & 7)) << 4);
 }
 
+// The keys of a request: [0, keep) and [first_key, kv_len), and its chunks, numbered from
+// first_split to n_splits with those between the kept ones and the window's left out.
 struct TdRange {
-    int kv_len, first_key, first_split, n_splits;
+    int kv_len, first_key, keep, first_split, n_splits, n_keep, gap;
+    __device__ __forceinline__ int chunk_of(int split) const { return split < n_keep ? split : split + gap; }
+    __device__ __forceinline__ bool sees(int key) const {
+        return key < kv_len && (key >= first_key || key < keep);
+    }
+    // whether a page holds keys that are read
+    __device__ __forceinline__ bool needs(int page, int page_size) const {
+        const int p0 = page * page_size;
+        return p0 < kv_len && (p0 + page_size > first_key || p0 < keep);
+    }
 };
-__device__ __forceinline__ TdRange td_range(int ctx_len, int window) {
+__device__ __forceinline__ TdRange td_range(int ctx_len, int window, int keep) {
     TdRange r;
     r.kv_len = ctx_len + 1;
     r.first_key = first_visible_key(ctx_len, window);
-    r.first_split = r.first_key / kTdChunk;
-    r.n_splits = (r.kv_len + kTdChunk - 1) / kTdChunk;
+    r.keep = keep;
+    const KeptSplits k = kept_splits(r.first_key, r.kv_len, keep, kTdChunk);
+    r.first_split = k.first;
+    r.n_splits = k.end;
+    r.n_keep = k.n_keep;
+    r.gap = k.gap;
     return r;
 }
 
@@ -51,7 +74,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map,
                         int req_base, long long k_row0, long long v_row0,
                         const int* __restrict__ block_table, int bt_stride,
                         const int* __restrict__ ctx_len, int nq, int nkv, int page_size,
-                        float scale_log2e, int window, float* __restrict__ part_o,
+                        float scale_log2e, int window, int keep, int maps, float* __restrict__ part_o,
                         float* __restrict__ part_ml, int max_splits, int merge_all,
                         __nv_bfloat16* __restrict__ out) {
     constexpr int CPR = HD / 8;
@@ -76,21 +99,19 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map,
 
     const int split = blockIdx.x, kvh = blockIdx.y, i = blockIdx.z;
     const int req = req_base + i, row = row_base + i;
-    const int G = nq / nkv;
-    const TdRange rg = td_range(ld_step(ctx_len + req), window);      // before the wait
+    const int G = nq / nkv * maps;                                    // MMA rows in use
+    const TdRange rg = td_range(ld_step(ctx_len + req), window, keep);      // before the wait
     if (split < rg.first_split || split >= rg.n_splits) {
         pdl_wait();
         return;
     }
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int k0 = split * kTdChunk;
+    const int k0 = rg.chunk_of(split) * kTdChunk;
     const int* bt = block_table + static_cast<size_t>(req) * bt_stride;
     const uint32_t bar_k = smem_u32(&bars[0]), bar_v = smem_u32(&bars[1]);
 
     // pages of this chunk that hold keys the request reads
     const int pages_in_chunk = kTdChunk / page_size;
-    const int first_page = max(k0, rg.first_key) / page_size;             // absolute index
-    const int last_page = (min(k0 + kTdChunk, rg.kv_len) - 1) / page_size;
     const int chunk_page0 = k0 / page_size;
     const int newest_page = (rg.kv_len - 1) / page_size;                  // written by the predecessor
 
@@ -98,18 +119,19 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map,
     // counts, then one lane per page looks its page up and issues that page's copies, so the
     // page-table reads run side by side instead of one after another.
     if (warp == 0) {
+        const unsigned used = __ballot_sync(0xffffffffu, lane < pages_in_chunk && rg.needs(chunk_page0 + lane, page_size));
         if (lane == 0) {
             mbar_init(bar_k, 1);
             mbar_init(bar_v, 1);
             mbar_fence_init();
-            const uint32_t bytes = static_cast<uint32_t>(last_page - first_page + 1) * page_size * HD * 2;
+            const uint32_t bytes = static_cast<uint32_t>(__popc(used)) * page_size * HD * 2;
             mbar_expect_tx(bar_k, bytes);
             mbar_expect_tx(bar_v, bytes);
         }
         __syncwarp();
         for (int p = lane; p < pages_in_chunk; p += 32) {
             const int ap = chunk_page0 + p;
-            if (ap < first_page || ap > last_page || ap == newest_page) continue;
+            if (!rg.needs(ap, page_size) || ap == newest_page) continue;
             const long long prow = (static_cast<long long>(ld_step(bt + ap)) * nkv + kvh) * page_size;
             const int r = p * page_size;
 #pragma unroll
@@ -125,15 +147,15 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map,
     // V rows of pages that are not loaded must not hold stale non-finite bit patterns
     for (int p = 0; p < pages_in_chunk; ++p) {
         const int ap = chunk_page0 + p;
-        if (ap >= first_page && ap <= last_page) continue;
+        if (rg.needs(ap, page_size)) continue;
         for (int c = tid; c < page_size * CPR; c += kTdThreads) {
             const int r = p * page_size + c / CPR, ch = c % CPR;
             *reinterpret_cast<uint4*>(Vs + tma_tile_offset(r, ch)) = make_uint4(0, 0, 0, 0);
         }
     }
     pdl_wait();
-    if (warp == 0 && newest_page >= max(first_page, chunk_page0) &&
-        newest_page <= last_page && lane == (newest_page - chunk_page0) % 32) {
+    if (warp == 0 && newest_page >= chunk_page0 && newest_page < chunk_page0 + pages_in_chunk &&
+        lane == newest_page - chunk_page0) {
         const int p = newest_page - chunk_page0;
         const long long prow = (static_cast<long long>(ld_step(bt + newest_page)) * nkv + kvh) * page_size;
         const int r = p * page_size;
@@ -147,11 +169,11 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map,
                         static_cast<int>(v_row0 + prow), bar_v);
     }
     // Q: rows of the group's heads, zero rows up to 16
-    const __nv_bfloat16* qrow = qkv + static_cast<size_t>(row) * row_stride + static_cast<size_t>(kvh) * G * HD;
+    const __nv_bfloat16* qrow = qkv + static_cast<size_t>(row) * row_stride + static_cast<size_t>(kvh) * (nq / nkv) * HD;
     for (int c = tid; c < kTdRows * CPR; c += kTdThreads) {
         const int r = c / CPR, ch = c - r * CPR;
-        const bool ok = r < G;
-        cp_async_16(smem_u32(Qs + swizzled_offset<HD>(r, ch)), ok ? qrow + r * HD + ch * 8 : qrow,
+        const bool ok = r < G && (maps == 1 || (ch >= CPR / 2) == (r & 1));
+        cp_async_16(smem_u32(Qs + swizzled_offset<HD>(r, ch)), ok ? qrow + (r >> (maps - 1)) * HD + ch * 8 : qrow,
                     ok ? 16 : 0);
     }
     cp_async_commit();
@@ -188,7 +210,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map,
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int key = k0 + kw + nt * 8 + (lane & 3) * 2 + (e & 1);
-            const bool ok = key < rg.kv_len && key >= rg.first_key;
+            const bool ok = rg.sees(key);
             const float v = ok ? s[nt][e] * scale_log2e : -INFINITY;
             s[nt][e] = v;
             if (e < 2) m_lo = fmaxf(m_lo, v); else m_hi = fmaxf(m_hi, v);
@@ -270,7 +292,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map,
                 *reinterpret_cast<uint32_t*>(dst + nt * 8 + (lane & 3) * 2) =
                     pack_bf16(o[nt][half * 2] * inv, o[nt][half * 2 + 1] * inv);
         } else {
-            const size_t p = (static_cast<size_t>(i) * nq + head) * max_splits + split;
+            const size_t p = (static_cast<size_t>(i) * nq * maps + head) * max_splits + split;
             float* dst = part_o + p * HD + warp * DW;
 #pragma unroll
             for (int nt = 0; nt < DW / 8; ++nt)
@@ -306,7 +328,7 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
                          int req_base, long long k_row0, long long v_row0,
                          const int* __restrict__ block_table, int bt_stride,
                          const int* __restrict__ ctx_len, int nq, int nkv, int page_size,
-                         float scale_log2e, int window, float* __restrict__ part_o,
+                         float scale_log2e, int window, int keep, int maps, float* __restrict__ part_o,
                          float* __restrict__ part_ml, int max_splits, int cpc, int merge_all,
                          __nv_bfloat16* __restrict__ out) {
     constexpr int CPR = HD / 8;
@@ -326,8 +348,8 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
 
     const int group = blockIdx.x, kvh = blockIdx.y, i = blockIdx.z;
     const int req = req_base + i, row = row_base + i;
-    const int G = nq / nkv;
-    const TdRange rg = td_range(ld_step(ctx_len + req), window);      // before the wait
+    const int G = nq / nkv * maps;                                    // MMA rows in use
+    const TdRange rg = td_range(ld_step(ctx_len + req), window, keep);      // before the wait
     const int c_begin = max(group * cpc, rg.first_split);
     const int c_end = min((group + 1) * cpc, rg.n_splits);
     if (c_begin >= c_end) {
@@ -340,11 +362,8 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
     const int pages_in_chunk = kTdChunk / page_size;
     const int newest_page = (rg.kv_len - 1) / page_size;   // written by the kernel before this one
 
-    // pages of chunk c (counted from c_begin) that hold keys the request reads
-    auto first_page_of = [&](int c) { return max((c_begin + c) * kTdChunk, rg.first_key) / page_size; };
-    auto last_page_of = [&](int c) {
-        return (min((c_begin + c + 1) * kTdChunk, rg.kv_len) - 1) / page_size;
-    };
+    // the first page of chunk c (counted from c_begin)
+    auto page0_of = [&](int c) { return rg.chunk_of(c_begin + c) * pages_in_chunk; };
     if (tid == 0) {
         for (int x = 0; x < kRingK; ++x) {
             mbar_init(smem_u32(&k_full[x]), 1);
@@ -360,10 +379,8 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
     // copied must not hold stale non-finite bit patterns (later they hold an older chunk's values,
     // which meet probabilities of zero).
     for (int c = 0; c < min(n_chunks, kRingV); ++c) {
-        const int fp = first_page_of(c), lp = last_page_of(c);
         for (int pg = 0; pg < pages_in_chunk; ++pg) {
-            const int ap = (c_begin + c) * pages_in_chunk + pg;
-            if (ap >= fp && ap <= lp) continue;
+            if (rg.needs(page0_of(c) + pg, page_size)) continue;
             for (int x = tid; x < page_size * CPR; x += kRingThreads) {
                 const int r = pg * page_size + x / CPR, ch = x % CPR;
                 *reinterpret_cast<uint4*>(Vs + c * TILE + tma_tile_offset(r, ch)) = make_uint4(0, 0, 0, 0);
@@ -391,13 +408,14 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
                 if (lane == 0) atomicExch(&g_decode_tma_error, 1);
                 break;
             }
-            const int fp = first_page_of(c), lp = last_page_of(c);
+            const int page0 = page0_of(c);
+            const int ap = page0 + lane;
+            const bool mine = lane < pages_in_chunk && rg.needs(ap, page_size);
+            const unsigned used = __ballot_sync(0xffffffffu, mine);
             if (lane == 0)
-                mbar_expect_tx(smem_u32(&full[st]), static_cast<uint32_t>(lp - fp + 1) * page_size * HD * 2);
+                mbar_expect_tx(smem_u32(&full[st]), static_cast<uint32_t>(__popc(used)) * page_size * HD * 2);
             __syncwarp();
-            const int ap = (c_begin + c) * pages_in_chunk + lane;
-            const bool mine = lane < pages_in_chunk && ap >= fp && ap <= lp;
-            const bool has_newest = newest_page >= fp && newest_page <= lp;
+            const bool has_newest = newest_page >= page0 && newest_page < page0 + pages_in_chunk;
             auto copy = [&]() {
                 const long long prow = (static_cast<long long>(ld_step(bt + ap)) * nkv + kvh) * page_size;
                 unsigned char* dst = tiles + st * TILE + lane * page_size * 128;
@@ -418,11 +436,11 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
 
     // ---- computing warps
     pdl_wait();
-    const __nv_bfloat16* qrow = qkv + static_cast<size_t>(row) * row_stride + static_cast<size_t>(kvh) * G * HD;
+    const __nv_bfloat16* qrow = qkv + static_cast<size_t>(row) * row_stride + static_cast<size_t>(kvh) * (nq / nkv) * HD;
     for (int c = tid; c < kTdRows * CPR; c += kTdThreads) {
         const int r = c / CPR, ch = c - r * CPR;
-        const bool ok = r < G;
-        cp_async_16(smem_u32(Qs + swizzled_offset<HD>(r, ch)), ok ? qrow + r * HD + ch * 8 : qrow,
+        const bool ok = r < G && (maps == 1 || (ch >= CPR / 2) == (r & 1));
+        cp_async_16(smem_u32(Qs + swizzled_offset<HD>(r, ch)), ok ? qrow + (r >> (maps - 1)) * HD + ch * 8 : qrow,
                     ok ? 16 : 0);
     }
     cp_async_commit();
@@ -443,7 +461,7 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
     for (int c = 0; c < n_chunks; ++c) {
         const unsigned char* Kt = Ks + (c % kRingK) * TILE;
         const unsigned char* Vt = Vs + (c % kRingV) * TILE;
-        const int k0 = (c_begin + c) * kTdChunk;
+        const int k0 = rg.chunk_of(c_begin + c) * kTdChunk;
         ok_wait = mbar_wait(smem_u32(&k_full[c % kRingK]), (c / kRingK) & 1) && ok_wait;
         // ---- S = Q K^T for this warp's 32 keys
         float s[4][4];
@@ -472,7 +490,7 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int key = k0 + kw + nt * 8 + (lane & 3) * 2 + (e & 1);
-                const bool ok = key < rg.kv_len && key >= rg.first_key;
+                const bool ok = rg.sees(key);
                 const float v = ok ? s[nt][e] * scale_log2e : -INFINITY;
                 s[nt][e] = v;
                 if (e < 2) m_lo = fmaxf(m_lo, v); else m_hi = fmaxf(m_hi, v);
@@ -560,7 +578,7 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
                 *reinterpret_cast<uint32_t*>(dst + nt * 8 + (lane & 3) * 2) =
                     pack_bf16(o[nt][half * 2] * inv, o[nt][half * 2 + 1] * inv);
         } else {
-            const size_t p = (static_cast<size_t>(i) * nq + head) * max_splits + group;
+            const size_t p = (static_cast<size_t>(i) * nq * maps + head) * max_splits + group;
             float* dst = part_o + p * HD + warp * DW;
 #pragma unroll
             for (int nt = 0; nt < DW / 8; ++nt)
@@ -576,9 +594,11 @@ int launch_tma_decode(const CUtensorMap* map, const void* qkv, int row_stride, i
                       const int* block_table, int bt_stride, const int* ctx_len, int nq, int nkv,
                       int page_size, float scale, int window, float* part_o, float* part_ml,
                       int max_splits, void* out, cudaStream_t stream, const float* sinks,
-                      const float* turn) {
-    // sinks and turned outputs are the merge kernel's: every request goes through it then
-    const int merge_all = sinks != nullptr || turn != nullptr;
+                      const float* turn, int keep = 0, const TwoMaps* two = nullptr) {
+    // sinks, turned outputs and differences of maps are the merge kernel's: every request goes
+    // through it then
+    const int merge_all = sinks != nullptr || turn != nullptr || two != nullptr;
+    const int maps = two != nullptr ? 2 : 1;
     constexpr int TILE = (HD / 64) * kHalfBytes;
     const size_t smem = 2 * TILE + kTdRows * HD * 2 + kTdRows * kTdChunk * 2 + 1024;
     cudaFuncSetAttribute(paged_decode_tma_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -604,9 +624,13 @@ int launch_tma_decode(const CUtensorMap* map, const void* qkv, int row_stride, i
         launch_pdl(paged_decode_ring_kernel<HD>, dim3(groups, nkv, n_decode), dim3(kRingThreads),
                    ring_smem, stream, *map, static_cast<const __nv_bfloat16*>(qkv), row_stride,
                    row_base, req_base, k_row0, v_row0, block_table, bt_stride, ctx_len, nq, nkv,
-                   page_size, scale * 1.4426950408889634f, window, part_o, part_ml, max_splits, cpc,
-                   merge_all, static_cast<__nv_bfloat16*>(out));
+                   page_size, scale * 1.4426950408889634f, window, keep, maps, part_o, part_ml, max_splits,
+                   cpc, merge_all, static_cast<__nv_bfloat16*>(out));
         int rc = launch_status();
+        if (rc == 0 && two != nullptr)
+            return launch_two_map_merge<HD>(part_o, part_ml, max_splits, kTdChunk, cpc, ctx_len, row_base,
+                                            req_base, n_decode, nq, window, keep, *two,
+                                            static_cast<__nv_bfloat16*>(out), stream);
         if (rc != 0 || (groups == 1 && !merge_all)) return rc;
         return launch_decode_merge<HD>(part_o, part_ml, max_splits, kTdChunk * cpc, ctx_len, row_base,
                                        req_base, n_decode, nq, window,
@@ -616,9 +640,13 @@ int launch_tma_decode(const CUtensorMap* map, const void* qkv, int row_stride, i
     launch_pdl(paged_decode_tma_kernel<HD>, dim3(grid), dim3(kTdThreads), smem, stream, 
         *map, static_cast<const __nv_bfloat16*>(qkv), row_stride, row_base, req_base, k_row0,
         v_row0, block_table, bt_stride, ctx_len, nq, nkv, page_size,
-        scale * 1.4426950408889634f, window, part_o, part_ml, max_splits, merge_all,
+        scale * 1.4426950408889634f, window, keep, maps, part_o, part_ml, max_splits, merge_all,
         static_cast<__nv_bfloat16*>(out));
     int rc = launch_status();
+    if (rc == 0 && two != nullptr)
+        return launch_two_map_merge<HD>(part_o, part_ml, max_splits, kTdChunk, 1, ctx_len, row_base, req_base,
+                                        n_decode, nq, window, keep, *two, static_cast<__nv_bfloat16*>(out),
+                                        stream);
     if (rc != 0 || (max_splits == 1 && !merge_all)) return rc;
     return launch_decode_merge<HD>(part_o, part_ml, max_splits, kTdChunk, ctx_len, row_base, req_base,
                                    n_decode, nq, window, static_cast<__nv_bfloat16*>(out), stream, sinks,
@@ -676,4 +704,33 @@ SOMI_API int somi_paged_attention_decode_tma(
     return launch_tma_decode<128>(map, qkv, row_stride, row_base, req_base, n_decode, k_row0,
                                   v_row0, block_table, bt_stride, ctx_len, nq, nkv, page_size,
                                   scale, window, part_o, part_ml, max_splits, out, stream, sinks, turn);
+}
+
+// Attention in two maps (two_maps.cuh) of single-token requests.  hd: the width of a value and of the
+// two keys of a head together.  part_o: float32 [n_decode, 2 nq, max_splits, hd], part_ml [.., 2], where
+// max_splits counts the chunks of 128 keys that a request reads at most, those between the kept
+// keys and the window left out.
+SOMI_API int somi_two_map_decode_supported(int nq, int nkv, int hd, int page_size) {
+    return somi_decode_tma_supported(2 * nq, nkv, hd, page_size);
+}
+SOMI_API int somi_two_map_attention_decode(
+    const void* tensor_map, const void* qkv, int row_stride, int row_base, int req_base,
+    int n_decode, long long k_row0, long long v_row0, const int* block_table, int bt_stride,
+    const int* ctx_len, int nq, int nkv, int hd, int page_size, float scale, int window, int keep,
+    float factor, float eps, float gain, const void* gate, long long gate_stride, float* part_o,
+    float* part_ml, int max_splits, void* out, cudaStream_t stream) {
+    if (n_decode <= 0) return 0;
+    if (!somi_two_map_decode_supported(nq, nkv, hd, page_size) || max_splits <= 0 || window < 0 ||
+        keep < 0 || n_decode > 65535 || nkv > 65535 || nq > 65535)
+        return SOMI_ERR_UNSUPPORTED;
+    const CUtensorMap* map = static_cast<const CUtensorMap*>(tensor_map);
+    const TwoMaps two{factor, eps, gain, gate, gate_stride};
+    if (hd == 64)
+        return launch_tma_decode<64>(map, qkv, row_stride, row_base, req_base, n_decode, k_row0,
+                                     v_row0, block_table, bt_stride, ctx_len, nq, nkv, page_size, scale,
+                                     window, part_o, part_ml, max_splits, out, stream, nullptr, nullptr,
+                                     keep, &two);
+    return launch_tma_decode<128>(map, qkv, row_stride, row_base, req_base, n_decode, k_row0, v_row0,
+                                  block_table, bt_stride, ctx_len, nq, nkv, page_size, scale, window,
+                                  part_o, part_ml, max_splits, out, stream, nullptr, nullptr, keep, &two);
 }

@@ -5,7 +5,10 @@
 // output may be multiplied by sigmoid(gate) in the epilogue (a logit per output element, or with
 // `gate_per_head` one per token and head).  `softcap` > 0: a score s becomes
 // softcap * tanh(s / softcap) before the softmax.  `sinks`: a score per query head that joins the
-// softmax's denominator without a key or a value (0 gives "one more in the denominator").
+// softmax's denominator without a key or a value (0 gives "one more in the denominator").  `keep`: beside a
+// window, the keys at positions below `keep` stay visible to all later tokens.  `maps`: a key/value
+// head holds that many keys of `hd` elements side by side in one cache row; query head i reads key
+// i % maps of key/value head i / (nq / nkv) (maps neighbouring query heads share a value head's keys).
 // It is the float32 path's attention and the fallback of the bfloat16 path for
 // sizes that the tensor-core kernels refuse.  Products are accumulated with
 // float32 FMAs, softmax is float32 and online, key tiles are aligned to
@@ -26,7 +29,7 @@ constexpr int kThreads = 128;
 constexpr int kMaxHd = 256;
 constexpr int kAccPerThread = kBM * kMaxHd / kThreads;   // 32
 
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(kThreads)
 paged_attention_generic_kernel(const T* __restrict__ qkv, int row_stride,
                                const T* __restrict__ kcache, const T* __restrict__ vcache,
@@ -36,7 +39,8 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int row_stride,
                                int n_prefill_tok, int nq, int nkv, int hd, int vd, int page_size,
                                float scale, int window, int chunk, const T* __restrict__ gate,
                                long long gate_stride, int gate_per_head, float softcap,
-                               const float* __restrict__ sinks, T* __restrict__ out) {
+                               const float* __restrict__ sinks, int keep, int maps,
+                               TO* __restrict__ out) {
     extern __shared__ float smem[];
     pdl_launch_dependents();
     pdl_wait();
@@ -60,7 +64,7 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int row_stride,
         rows = 1;
     }
     const int head = blockIdx.y;
-    const int kvh = head / (nq / nkv);
+    const int kvh = head / (nq / nkv), map = head % maps;
     const int tid = threadIdx.x;
     const int q_pos0 = ctx_len[req] + (row0 - cu_q[req]);
     const int kv_end = q_pos0 + rows;                                   // exclusive
@@ -79,14 +83,17 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int row_stride,
     for (int i = 0; i < kAccPerThread; ++i) acc[i] = 0.f;
     __syncthreads();
 
-    for (int kb = (kv_first / kBN) * kBN; kb < kv_end; kb += kBN) {
+    const int kb_first = (kv_first / kBN) * kBN;
+    // tiles of kept keys in front of the window's, then the window's
+    for (int kb = keep > 0 ? 0 : kb_first; kb < kv_end; kb += kBN) {
+        if (kb >= keep && kb < kb_first) kb = kb_first;
         for (int idx = tid; idx < kBN * hd; idx += kThreads) {
             const int n = idx / hd, d = idx - n * hd;
             const int j = kb + n;
             float kval = 0.f;
-            if (j >= kv_first && j < kv_end) {
+            if ((j >= kv_first || j < keep) && j < kv_end) {
                 const int page = bt[j / page_size];
-                kval = to_float(kcache[((static_cast<size_t>(page) * nkv + kvh) * page_size + j % page_size) * hd + d]);
+                kval = to_float(kcache[(((static_cast<size_t>(page) * nkv + kvh) * page_size + j % page_size) * maps + map) * hd + d]);
             }
             Ks[n * (hd + 1) + d] = kval;
         }
@@ -94,7 +101,7 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int row_stride,
             const int n = idx / vd, d = idx - n * vd;
             const int j = kb + n;
             float vval = 0.f;
-            if (j >= kv_first && j < kv_end) {
+            if ((j >= kv_first || j < keep) && j < kv_end) {
                 const int page = bt[j / page_size];
                 vval = to_float(vcache[((static_cast<size_t>(page) * nkv + kvh) * page_size + j % page_size) * vd + d]);
             }
@@ -105,8 +112,9 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int row_stride,
             const int m = idx / kBN, n = idx - m * kBN;
             const int j = kb + n, qp = q_pos0 + m;
             float s = -INFINITY;
-            if (m < rows && j <= qp && j >= kv_first && (window <= 0 || j > qp - window) &&
-                (chunk <= 0 || j / chunk == qp / chunk)) {
+            if (m < rows && j <= qp &&
+                (j < keep || (j >= kv_first && (window <= 0 || j > qp - window) &&
+                              (chunk <= 0 || j / chunk == qp / chunk)))) {
                 s = 0.f;
                 const float* q = Qs + m * hd;
                 const float* k = Ks + n * (hd + 1);
@@ -164,7 +172,7 @@ paged_attention_generic_kernel(const T* __restrict__ qkv, int row_stride,
                                                   (gate_per_head ? head : head * vd + d)]);
                     o = o / (1.0f + expf(-z));
                 }
-                out[static_cast<size_t>(row0 + m) * (nq * vd) + head * vd + d] = from_float<T>(o);
+                out[static_cast<size_t>(row0 + m) * (nq * vd) + head * vd + d] = from_float<TO>(o);
             }
         }
     }
@@ -230,28 +238,30 @@ SOMI_API int somi_paged_attention_generic(
     const int* block_table, int bt_stride, const int* cu_q, const int* ctx_len, const int* tiles,
     int n_tiles, int n_prefill_req, int n_prefill_tok, int n_decode, int nq, int nkv, int hd, int vd,
     int page_size, float scale, int window, int chunk, const void* gate, long long gate_stride,
-    int gate_per_head, float softcap, const float* sinks, void* out, cudaStream_t stream) {
+    int gate_per_head, float softcap, const float* sinks, int keep, int maps, int out_f32, void* out,
+    cudaStream_t stream) {
     if (n_tiles + n_decode <= 0) return 0;
     if (hd <= 0 || hd > kMaxHd || vd <= 0 || vd > kMaxHd || nkv <= 0 || nq % nkv || page_size <= 0 ||
-        (window > 0 && chunk > 0))
+        (window > 0 && chunk > 0) || keep < 0 || (keep > 0 && window <= 0) || maps <= 0 || (nq / nkv) % maps)
         return SOMI_ERR_UNSUPPORTED;
     const size_t smem = sizeof(float) * (static_cast<size_t>(kBM) * hd + kBN * (hd + 1) + kBN * vd +
                                          kBM * (kBN + 1) + 3 * kBM);
     dim3 grid(n_tiles + n_decode, nq);
-#define SOMI_LAUNCH_ATT(T)                                                                      \
+#define SOMI_LAUNCH_ATT(T, TO)                                                                  \
     do {                                                                                        \
         if (smem > 48 * 1024)                                                                   \
-            cudaFuncSetAttribute(paged_attention_generic_kernel<T>,                             \
+            cudaFuncSetAttribute(paged_attention_generic_kernel<T, TO>,                         \
                                  cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
-        launch_pdl(paged_attention_generic_kernel<T>, dim3(grid), dim3(kThreads), smem, stream,                     \
+        launch_pdl(paged_attention_generic_kernel<T, TO>, dim3(grid), dim3(kThreads), smem, stream,                     \
             static_cast<const T*>(qkv), row_stride, static_cast<const T*>(kcache),              \
             static_cast<const T*>(vcache), block_table, bt_stride, cu_q, ctx_len, tiles,        \
             n_tiles, n_prefill_req, n_prefill_tok, nq, nkv, hd, vd, page_size, scale, window,   \
             chunk, static_cast<const T*>(gate), gate_stride, gate_per_head, softcap, sinks,     \
-            static_cast<T*>(out));                                                              \
+            keep, maps, static_cast<TO*>(out));                                                              \
     } while (0)
-    if (dtype == SOMI_F32) SOMI_LAUNCH_ATT(float);
-    else SOMI_LAUNCH_ATT(__nv_bfloat16);
+    if (dtype == SOMI_F32) SOMI_LAUNCH_ATT(float, float);
+    else if (out_f32) SOMI_LAUNCH_ATT(__nv_bfloat16, float);
+    else SOMI_LAUNCH_ATT(__nv_bfloat16, __nv_bfloat16);
 #undef SOMI_LAUNCH_ATT
     return launch_status();
 }

@@ -34,9 +34,18 @@
 // value producer, warp 11 idle.  Two key stages and three value stages at head size 128 (a value
 // tile is read a round later than the key tile that came with it), four and four at 64.
 //
+// With `TWO_MAPS` (attention in two maps, two_maps.cuh) the CTA's two query tiles are the two queries
+// of the same 128 rows: a key row of HD elements holds the keys of both maps, map x being its half
+// x, so the keys of both maps arrive in one tile and the values are fetched once for both.  Both
+// tiles then have the same rows, positions and key tiles; at the end each softmax warp group takes
+// half of the head's columns of both outputs, and the difference of the maps, its norm and the
+// gate are made from the float32 accumulators.  There first tokens may stay visible beside a
+// window (`keep`): the key tiles that hold them come in front of the window's.
+//
 // The reference's prefill kernel (somi_inference/core/flash_attention_triton.py:31-194) is a
 // FlashAttention-2 loop on `tl.dot`; formulas in somi_inference/models/qwen2.py:158-186.
 #include "tcgen05.cuh"
+#include "two_maps.cuh"
 
 namespace somi {
 
@@ -54,7 +63,7 @@ constexpr int kPpKvHalf = kPpBN * 128;
 
 __device__ int g_prefill_pp_error = 0;
 
-template <int HD>
+template <int HD, bool TWO_MAPS>
 __global__ void __launch_bounds__(kPpThreads, 1)
 paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
                         const __grid_constant__ CUtensorMap kv_map, long long k_row0,
@@ -63,7 +72,7 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
                         const int* __restrict__ tiles, int nq, int nkv, int page_size,
                         float scale_log2e, int window, const float* __restrict__ sinks,
                         const float2* __restrict__ turn, __nv_bfloat16* __restrict__ out,
-                        int n_q_tiles) {
+                        int n_q_tiles, int keep, TwoMaps two) {
     constexpr int HALVES = HD / 64;
     constexpr int QTILE = HALVES * kPpQHalf;
     constexpr int TILE = HALVES * kPpKvHalf;
@@ -72,13 +81,14 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
     extern __shared__ unsigned char smem_raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>(
         (reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
-    unsigned char* Qs = base;                            // two query tiles
-    unsigned char* Ks = Qs + 2 * QTILE;                  // KST tiles
+    unsigned char* Qs = base;                            // two query tiles (two maps: one)
+    unsigned char* Ks = Qs + (TWO_MAPS ? 1 : 2) * QTILE;                  // KST tiles
     unsigned char* Vs = Ks + KST * TILE;                 // VST tiles
     __shared__ __align__(8) unsigned long long q_full[2], k_full[kPpMaxStages], k_empty[kPpMaxStages],
         v_full[kPpMaxStages], v_empty[kPpMaxStages], s_full[2], p_full[2], o_done[2], v_zeroed;
     __shared__ uint32_t tmem_base_s;
     __shared__ int failed_s;
+    __shared__ float map_scale_s[TWO_MAPS ? 2 : 1][kPpBM], map_square_s[TWO_MAPS ? 2 : 1][kPpBM];
 
     pdl_launch_dependents();
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -120,13 +130,16 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
     const int req = tiles[3 * tile], row0 = tiles[3 * tile + 1];
     const int rows = tiles[3 * tile + 2];
     const int head = rank % nq, kvh = head / (nq / nkv);
-    const bool has_b = rows > kPpBM;
+    const bool has_b = TWO_MAPS || rows > kPpBM;
     const int q_pos0 = ctx_len[req] + (row0 - cu_q[req]);
     const int kv_first = first_visible_key(q_pos0, window);
     const int kb0 = (kv_first / kPpBN) * kPpBN;
     const int end_a = q_pos0 + min(rows, kPpBM), end_all = q_pos0 + rows;
-    const int n_a = (end_a - kb0 + kPpBN - 1) / kPpBN;            // key tiles that tile A reads
-    const int n_t = (end_all - kb0 + kPpBN - 1) / kPpBN;          // key tiles of the CTA
+    // tiles of kept keys in front of the window's
+    const int n_pre = TWO_MAPS && keep > 0 ? min((keep + kPpBN - 1) / kPpBN, kb0 / kPpBN) : 0;
+    const int n_a = n_pre + (end_a - kb0 + kPpBN - 1) / kPpBN;    // key tiles that tile A reads
+    const int n_t = n_pre + (end_all - kb0 + kPpBN - 1) / kPpBN;  // key tiles of the CTA
+    auto key_tile = [&](int t) { return t < n_pre ? t * kPpBN : kb0 + (t - n_pre) * kPpBN; };
     const int* bt = block_table + static_cast<size_t>(req) * bt_stride;
 
     // The softmax threads hold a row of 128 scores in registers; the producer and issuing warps
@@ -141,7 +154,7 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
         // ---- producer warps, one for the keys (and Q) and one for the values.  Lane 0 keeps the
         // barriers, one lane per page looks its page up and issues that page's copies.
         if (warp == 8 && lane == 0) {
-            for (int x = 0; x < (has_b ? 2 : 1); ++x) {
+            for (int x = 0; x < (has_b && !TWO_MAPS ? 2 : 1); ++x) {
                 mbar_expect_tx(smem_u32(&q_full[x]), kPpBM * HD * 2);
 #pragma unroll
                 for (int h = 0; h < HALVES; ++h)
@@ -157,17 +170,22 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
         __syncwarp();
         for (int t = 0; t < n_t; ++t) {
             const int st = t % n_st;
-            const int kb = kb0 + t * kPpBN;
+            const int kb = key_tile(t);
             const int p_lo = max(kb, kv_first) / page_size;
             const int p_hi = (min(kb + kPpBN, end_all) - 1) / page_size;
-            int my_page = -1;
+            int my_page = -1, n_pages = p_hi - p_lo + 1;
             const int ap = kb / page_size + lane;
-            if (lane < pages_per_tile && ap >= p_lo && ap <= p_hi) my_page = bt[ap];
+            bool mine = lane < pages_per_tile && ap >= p_lo && ap <= p_hi;
+            if constexpr (TWO_MAPS) {
+                mine = mine || (lane < pages_per_tile && ap <= p_hi && ap * page_size < keep);
+                n_pages = __popc(__ballot_sync(0xffffffffu, mine));
+            }
+            if (mine) my_page = bt[ap];
             const uint32_t bar = smem_u32(which ? &v_full[st] : &k_full[st]);
             int ok = 1;
             if (lane == 0) {
                 ok = mbar_wait(smem_u32(which ? &v_empty[st] : &k_empty[st]), ((t / n_st) & 1) ^ 1) ? 1 : 0;
-                if (ok) mbar_expect_tx(bar, static_cast<uint32_t>(p_hi - p_lo + 1) * page_size * HD * 2);
+                if (ok) mbar_expect_tx(bar, static_cast<uint32_t>(n_pages) * page_size * HD * 2);
                 else failed_s = 1;
             }
             ok = __shfl_sync(0xffffffffu, ok, 0);
@@ -211,13 +229,17 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
             };
             auto scores = [&](int x, int t) {            // S_x(t) = Q_x K(t)^T
                 const uint64_t kd = k_desc + (((t % KST) * TILE) >> 4);
-                const uint64_t qd = q_desc + ((x * QTILE) >> 4);
+                const uint64_t qd = q_desc + (TWO_MAPS ? 0 : (x * QTILE) >> 4);
+                // (two maps: query x and key x are half x of the rows)
+                const int first16 = TWO_MAPS ? x * (HD / 32) : 0;
 #pragma unroll
-                for (int k16 = 0; k16 < HD / 16; ++k16)
+                for (int i16 = 0; i16 < (TWO_MAPS ? HD / 32 : HD / 16); ++i16) {
+                    const int k16 = first16 + i16;
                     t5::mma_ss(tmem_s + x * kPpBN,
                                qd + (((k16 >> 2) * kPpQHalf + (k16 & 3) * 32) >> 4),
                                kd + (((k16 >> 2) * kPpKvHalf + (k16 & 3) * 32) >> 4), idesc_qk,
-                               k16 > 0 ? 1u : 0u);
+                               i16 > 0 ? 1u : 0u);
+                }
                 t5::commit(smem_u32(&s_full[x]));
             };
             auto outputs = [&](int x, int t) {           // O_x += P_x(t) V(t)
@@ -234,7 +256,7 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
             wait(&k_full[0], 0);
             if (ok) scores(0, 0);
             if (has_b) {
-                wait(&q_full[1], 0);
+                if (!TWO_MAPS) wait(&q_full[1], 0);
                 if (ok) scores(1, 0);
             }
             if (ok) t5::commit(smem_u32(&k_empty[0]));
@@ -280,12 +302,13 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
             const int q = warp & 3;                                  // lane quarter this warp may access
             const int row = q * 32 + lane;                           // row within the query tile
             const uint32_t lane_addr = static_cast<uint32_t>(q * 32) << 16;
-            const int tile_pos0 = q_pos0 + x * kPpBM;                // position of the tile's first row
+            const int tile_pos0 = q_pos0 + (TWO_MAPS ? 0 : x * kPpBM);   // position of the tile's first row
             const int pos = tile_pos0 + row;
             const int lo = first_visible_key(pos, window);
             // the highest first visible key among the tile's rows
             const int lo_max = first_visible_key(tile_pos0 + kPpBM - 1, window);
             const unsigned span = static_cast<unsigned>(pos - lo);
+            const int keep_end = TWO_MAPS ? min(keep, pos + 1) : 0;  // keys below it are visible, too
             const int n_x = x == 0 ? n_a : n_t;
             const uint32_t s_addr = tmem_s + x * kPpBN + lane_addr;
             const uint32_t o_addr = tmem_o + x * kPpBN + lane_addr;
@@ -305,9 +328,10 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
                 }
                 ok = mbar_wait(smem_u32(&s_full[x]), t & 1, ok ? 400000 : 1) && ok;
                 t5::fence_after();
-                const int kb = kb0 + t * kPpBN;
+                const int kb = key_tile(t);
                 // a tile in which no row of this query tile has a hidden key takes the short way
-                const bool tile_inner = kb + kPpBN - 1 <= tile_pos0 && kb >= lo_max;
+                const bool tile_inner = kb + kPpBN - 1 <= tile_pos0 &&
+                                        (kb >= lo_max || (TWO_MAPS && kb + kPpBN <= keep));
                 // ---- the row's 128 scores into registers: four loads in flight, one wait
                 uint32_t sv[128];
 #pragma unroll
@@ -323,7 +347,8 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
                     for (int j = 0; j < 128; ++j) {
                         // key in [lo, pos] as one unsigned comparison
                         const unsigned d = static_cast<unsigned>(kb + j - lo);
-                        const float v = d <= span ? __uint_as_float(sv[j]) : -INFINITY;
+                        const bool seen = d <= span || (TWO_MAPS && kb + j < keep_end);
+                        const float v = seen ? __uint_as_float(sv[j]) : -INFINITY;
                         sv[j] = __float_as_uint(v);
                         mx[j & 3] = fmaxf(mx[j & 3], v);
                     }
@@ -390,6 +415,48 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
             // ---- the output of this row
             ok = mbar_wait(smem_u32(&o_done[x]), 0, ok ? 400000 : 1) && ok;
             t5::fence_after();
+            if constexpr (TWO_MAPS) {
+                ok = mbar_wait(smem_u32(&o_done[x ^ 1]), 0, ok ? 400000 : 1) && ok;
+                t5::fence_after();
+                if (!ok) failed_s = 1;
+                map_scale_s[x][row] = (x == 0 ? 1.0f : -two.factor) / l;
+                asm volatile("bar.sync 1, 256;\n" ::: "memory");     // the two softmax warp groups
+                const float c0 = map_scale_s[0][row], c1 = map_scale_s[1][row];
+                const uint32_t col0 = x * (HD / 2);                  // this warp group's half of the head
+                const uint32_t a_addr = tmem_o + lane_addr + col0, b_addr = a_addr + kPpBN;
+                float dif[HD / 2];
+                float ss = 0.f;
+#pragma unroll
+                for (int c = 0; c < HD / 64; ++c) {
+                    uint32_t v[32], u[32];
+                    t5::ld32_nowait(a_addr + c * 32, v);
+                    t5::ld32_nowait(b_addr + c * 32, u);
+                    t5::wait_ld();
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) {
+                        const float y = fmaf(__uint_as_float(u[j]), c1, __uint_as_float(v[j]) * c0);
+                        dif[c * 32 + j] = y;
+                        ss = fmaf(y, y, ss);
+                    }
+                }
+                map_square_s[x][row] = ss;
+                asm volatile("bar.sync 1, 256;\n" ::: "memory");
+                if (row < rows) {
+                    const float mean = (map_square_s[0][row] + map_square_s[1][row]) / static_cast<float>(HD);
+                    const float f = two.gain / sqrtf(mean + two.eps) *
+                                    two_map_gate<__nv_bfloat16>(two, static_cast<size_t>(row0 + row), head);
+                    __nv_bfloat16* dst = out + static_cast<size_t>(row0 + row) * nq * HD + head * HD + col0;
+#pragma unroll
+                    for (int d = 0; d < HD / 2; d += 8) {
+                        uint4 w;
+                        w.x = pack_bf16(dif[d] * f, dif[d + 1] * f);
+                        w.y = pack_bf16(dif[d + 2] * f, dif[d + 3] * f);
+                        w.z = pack_bf16(dif[d + 4] * f, dif[d + 5] * f);
+                        w.w = pack_bf16(dif[d + 6] * f, dif[d + 7] * f);
+                        *reinterpret_cast<uint4*>(dst + d) = w;
+                    }
+                }
+            } else {
             if (!ok) failed_s = 1;
             // a sink: one more score in the denominator, without a value
             if (sinks != nullptr) l += fast_exp2(sinks[head] * 1.4426950408889634f - m);
@@ -449,6 +516,7 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
                     }
                 }
             }
+            }
         }
     }
     t5::fence_before();
@@ -461,21 +529,21 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
     if (tid == 0 && failed_s) atomicExch(&g_prefill_pp_error, 1);
 }
 
-template <int HD>
+template <int HD, bool TWO_MAPS = false>
 int launch_prefill_pp(const CUtensorMap* q_map, const CUtensorMap* kv_map, long long k_row0,
                       long long v_row0, const int* block_table, int bt_stride, const int* cu_q,
                       const int* ctx_len, const int* tiles, int n_tiles, int nq, int nkv,
                       int page_size, float scale, int window, const float* sinks, const float* turn,
-                      void* out, cudaStream_t stream) {
-    const size_t smem = 2 * (HD / 64) * kPpQHalf +
+                      void* out, cudaStream_t stream, int keep = 0, const TwoMaps& two = TwoMaps{}) {
+    const size_t smem = (TWO_MAPS ? 1 : 2) * (HD / 64) * kPpQHalf +
                         (pp_k_stages(HD) + pp_v_stages(HD)) * (HD / 64) * kPpKvHalf + 1024;
-    cudaFuncSetAttribute(paged_prefill_pp_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                         (int)smem);
+    cudaFuncSetAttribute(paged_prefill_pp_kernel<HD, TWO_MAPS>,
+                         cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     dim3 grid(static_cast<unsigned>(nq) * n_tiles);
-    launch_pdl(paged_prefill_pp_kernel<HD>, grid, dim3(kPpThreads), smem, stream, *q_map, *kv_map,
+    launch_pdl(paged_prefill_pp_kernel<HD, TWO_MAPS>, grid, dim3(kPpThreads), smem, stream, *q_map, *kv_map,
                k_row0, v_row0, block_table, bt_stride, cu_q, ctx_len, tiles, nq, nkv, page_size,
                scale * 1.4426950408889634f, window, sinks, reinterpret_cast<const float2*>(turn),
-               static_cast<__nv_bfloat16*>(out), n_tiles);
+               static_cast<__nv_bfloat16*>(out), n_tiles, keep, two);
     return launch_status();
 }
 
@@ -516,4 +584,26 @@ SOMI_API int somi_paged_attention_prefill_pp(
                                      stream);
     return launch_prefill_pp<128>(qm, km, k_row0, v_row0, block_table, bt_stride, cu_q, ctx_len, tiles,
                                   n_tiles, nq, nkv, page_size, scale, window, sinks, turn, out, stream);
+}
+
+// Attention in two maps (two_maps.cuh) of prompt portions.  hd (64 or 128): the width of a value and of
+// the two queries, or keys, of a head together.  `tiles`: as above with rows <= 128.
+SOMI_API int somi_two_map_attention_prefill(
+    const void* q_map, const void* kv_map, long long k_row0, long long v_row0,
+    const int* block_table, int bt_stride, const int* cu_q, const int* ctx_len, const int* tiles,
+    int n_tiles, int nq, int nkv, int hd, int page_size, float scale, int window, int keep, float factor,
+    float eps, float gain, const void* gate, long long gate_stride, void* out, cudaStream_t stream) {
+    if (n_tiles <= 0) return 0;
+    if (!somi_prefill_pp_supported(nq, nkv, hd, page_size) || window < 0 || keep < 0 || (keep > 0 && window == 0))
+        return SOMI_ERR_UNSUPPORTED;
+    const CUtensorMap* qm = static_cast<const CUtensorMap*>(q_map);
+    const CUtensorMap* km = static_cast<const CUtensorMap*>(kv_map);
+    const TwoMaps two{factor, eps, gain, gate, gate_stride};
+    if (hd == 64)
+        return launch_prefill_pp<64, true>(qm, km, k_row0, v_row0, block_table, bt_stride, cu_q, ctx_len,
+                                           tiles, n_tiles, nq, nkv, page_size, scale, window, nullptr,
+                                           nullptr, out, stream, keep, two);
+    return launch_prefill_pp<128, true>(qm, km, k_row0, v_row0, block_table, bt_stride, cu_q, ctx_len,
+                                        tiles, n_tiles, nq, nkv, page_size, scale, window, nullptr, nullptr,
+                                        out, stream, keep, two);
 }

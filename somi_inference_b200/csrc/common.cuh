@@ -82,6 +82,21 @@ __host__ __device__ __forceinline__ int first_visible_key(int pos, int window) {
     return 0;
 }
 
+// A gated activation: g * sigmoid(alpha * (g + cubic * g^3)) * (u + shift) with g = min(gate, limit) and
+// u = up within +-limit.  Limit infinite, alpha 1, shift 0, cubic 0: silu(gate) * up; alpha =
+// 2 sqrt(2 / pi), cubic 0.044715: gelu(gate) * up in gelu's tanh form, since (1 + tanh(y)) / 2 = sigmoid(2y).
+struct GluForm { float limit, alpha, shift, cubic; };
+
+// the argument of the sigmoid
+__device__ __forceinline__ float glu_argument(float g, const GluForm& f) {
+    return f.alpha * (f.cubic != 0.f ? fmaf(f.cubic * g * g, g, g) : g);
+}
+__device__ __forceinline__ float glu(float gate, float up, const GluForm& f) {
+    const float g = fminf(gate, f.limit);
+    const float u = fminf(fmaxf(up, -f.limit), f.limit);
+    return g / (1.0f + expf(-glu_argument(g, f))) * (u + f.shift);
+}
+
 inline int launch_status() { return static_cast<int>(cudaGetLastError()); }
 
 // ---- programmatic dependent launch

@@ -30,9 +30,6 @@ constexpr int kGemmWBytes = kGemmBN * kGemmBK * 2;      // 16 KiB
 
 enum GemmMode { kGemmBf16 = 0, kGemmF32 = 1, kGemmPartialF32 = 2, kGemmSwiGLU = 3, kGemmXieluSide = 4 };
 
-// the gated activation of kGemmSwiGLU (limit infinite, alpha 1, shift 0: silu(gate) * up)
-struct GluForm { float limit, alpha, shift; };
-
 __device__ int g_gemm_error = 0;
 
 __device__ __forceinline__ uint64_t umma_smem_desc(uint32_t smem_addr) {
@@ -267,7 +264,7 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap w_map,
                     }
                 }
             } else {   // kGemmSwiGLU: even rows of W are gate rows, odd rows the matching up rows;
-                // g * sigmoid(alpha g) * (u + shift), g = min(gate, limit), u = clamp(up, -limit, limit)
+                // the gated activation `glu` describes
                 __nv_bfloat16* y = static_cast<__nv_bfloat16*>(out);
                 const int half_n = N >> 1;
 #pragma unroll
@@ -278,7 +275,7 @@ skinny_gemm_kernel(const __grid_constant__ CUtensorMap w_map,
                         const float g = fminf(acc[m], glu.limit);
                         const float u = fminf(fmaxf(other, -glu.limit), glu.limit) + glu.shift;
                         y[static_cast<size_t>(m) * half_n + (n >> 1)] =
-                            __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-glu.alpha * g)) * u);
+                            __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-glu_argument(g, glu))) * u);
                     }
                 }
             }
@@ -346,18 +343,18 @@ SOMI_API int somi_gemm_error() {
 SOMI_API int somi_skinny_gemm_act(const void* w_map, const void* x_map, int x_box_rows, int M, int N,
                                   int K, int splits, int mode, const void* bias, int bias_dtype,
                                   void* out, void* out2, int n_act, const float* act, float limit,
-                                  float alpha, float shift, int deep_ring, cudaStream_t stream);
+                                  float alpha, float shift, float cubic, int deep_ring, cudaStream_t stream);
 
 // mode: 0 bf16 [M, N]; 1 float32 [M, N]; 2 float32 partial sums [splits, M, N] (bias in split 0);
 // 3 the gated activation (GluForm) over interleaved gate/up rows, bf16 [M, N / 2].  `x_box_rows` is the box height the
 // x tensor map was made with (16, 32 or 64) and must be >= M.
 SOMI_API int somi_skinny_gemm(const void* w_map, const void* x_map, int x_box_rows, int M, int N,
                               int K, int splits, int mode, const void* bias, int bias_dtype,
-                              void* out, float limit, float alpha, float shift, int deep_ring,
+                              void* out, float limit, float alpha, float shift, float cubic, int deep_ring,
                               cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     return somi_skinny_gemm_act(w_map, x_map, x_box_rows, M, N, K, splits, mode, bias, bias_dtype, out,
-                                nullptr, 0, nullptr, limit, alpha, shift, deep_ring, stream);
+                                nullptr, 0, nullptr, limit, alpha, shift, cubic, deep_ring, stream);
 }
 
 // The same with mode 4: xIELU (its two numbers in `act`, float32) of the first `n_act` features
@@ -365,7 +362,7 @@ SOMI_API int somi_skinny_gemm(const void* w_map, const void* x_map, int x_box_ro
 SOMI_API int somi_skinny_gemm_act(const void* w_map, const void* x_map, int x_box_rows, int M, int N,
                                   int K, int splits, int mode, const void* bias, int bias_dtype,
                                   void* out, void* out2, int n_act, const float* act, float limit,
-                                  float alpha, float shift, int deep_ring, cudaStream_t stream) {
+                                  float alpha, float shift, float cubic, int deep_ring, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (M > x_box_rows || K % 8 != 0 || K <= 0 || mode < 0 || mode > 4) return SOMI_ERR_UNSUPPORTED;
     if (mode == kGemmSwiGLU && (N & 1)) return SOMI_ERR_UNSUPPORTED;
@@ -380,7 +377,7 @@ SOMI_API int somi_skinny_gemm_act(const void* w_map, const void* x_map, int x_bo
     // and epilogue overlap the other's main loop.
 #define SOMI_SKINNY(TOK, ST) \
     return launch_skinny<TOK, ST>(wm, xm, M, N, K, splits, mode, bias, bias_dtype, out, stride, stream, \
-                                  out2, n_act, act, GluForm{limit, alpha, shift})
+                                  out2, n_act, act, GluForm{limit, alpha, shift, cubic})
     switch (x_box_rows) {
         case 16: if (deep_ring) SOMI_SKINNY(16, 8); else SOMI_SKINNY(16, 6);
         case 32: if (deep_ring) SOMI_SKINNY(32, 8); else SOMI_SKINNY(32, 4);

@@ -65,7 +65,8 @@ __global__ void embed_sinusoid_layernorm_kernel(const int* __restrict__ ids,
 
 // ------------------------------------------------ gated residual + layer norm
 // r = residual[row] + g * sum_s delta[s][row], g = sigmoid(gate[row]) (1 without a gate);
-// if write_back: residual[row] = r;  out[b] = (r - mean) * rstd * weight  (rms = 1: r * rrms * weight),
+// if write_back: residual[row] = r;  out[b] = (r - mean) * rstd * weight + bias  (rms = 1: r * rrms * weight
+// + bias; bias null: 0),
 // row = rows ? rows[b] : b.  delta: [splits] partial sums `split_stride` elements apart, added in order;
 // the gate's logits may be partial sums of the same kind.  `extra`: float32 rows [N, H] that are
 // added too, outside the gate (a second branch of the same layer).
@@ -77,7 +78,7 @@ __global__ void add_layernorm_kernel(float* __restrict__ residual, const TD* __r
                                      const void* __restrict__ weight, int weight_dtype, float eps,
                                      TO* __restrict__ out, const int* __restrict__ rows, int H,
                                      int write_back, int rms, int vec4,
-                                     const float* __restrict__ extra) {
+                                     const float* __restrict__ extra, const void* __restrict__ bias) {
     extern __shared__ __align__(16) float row_buf[];
     __shared__ float scratch[33];
     pdl_launch_dependents();
@@ -157,6 +158,11 @@ __global__ void add_layernorm_kernel(float* __restrict__ residual, const TD* __r
                 F4 y;
 #pragma unroll
                 for (int e = 0; e < 4; ++e) y.v[e] = (v[k].v[e] - mean) * rstd * w.v[e];
+                if (bias != nullptr) {
+                    const F4 c = load4_any(bias, weight_dtype, i);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) y.v[e] += c.v[e];
+                }
                 store4(o + i, y);
             }
         }
@@ -188,7 +194,8 @@ __global__ void add_layernorm_kernel(float* __restrict__ residual, const TD* __r
         mean_rstd(row_buf, H, eps, scratch, mean, rstd);
     }
     for (int i = threadIdx.x; i < H; i += blockDim.x)
-        o[i] = from_float<TO>((row_buf[i] - mean) * rstd * load_as_float(weight, weight_dtype, i));
+        o[i] = from_float<TO>((row_buf[i] - mean) * rstd * load_as_float(weight, weight_dtype, i) +
+                              (bias != nullptr ? load_as_float(bias, weight_dtype, i) : 0.f));
 }
 
 // ------------------------------------------------- short causal convolution
@@ -472,7 +479,8 @@ SOMI_API int somi_add_layernorm(float* residual, const void* delta, int delta_dt
                                 long long gate_stride, int gate_splits, long long gate_split_stride,
                                 const void* weight, int weight_dtype, float eps,
                                 void* out, int out_dtype, const int* rows, int n_out, int H,
-                                int write_back, int rms, const float* extra, cudaStream_t stream) {
+                                int write_back, int rms, const float* extra, const void* bias,
+                                cudaStream_t stream) {
     if (n_out <= 0) return 0;
     if (delta_splits < 1 || (delta_splits > 1 && delta_dtype != SOMI_F32)) return SOMI_ERR_UNSUPPORTED;
     if (gate && !delta) return SOMI_ERR_UNSUPPORTED;
@@ -484,7 +492,7 @@ SOMI_API int somi_add_layernorm(float* residual, const void* delta, int delta_dt
                      (gate_split_stride & 3) == 0 &&
                      ((reinterpret_cast<uintptr_t>(delta) | reinterpret_cast<uintptr_t>(gate) |
                        reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(weight) |
-                       reinterpret_cast<uintptr_t>(extra)) & 15) == 0;
+                       reinterpret_cast<uintptr_t>(extra) | reinterpret_cast<uintptr_t>(bias)) & 15) == 0;
     if (extra != nullptr && delta == nullptr) return SOMI_ERR_UNSUPPORTED;
     // few rows (a decode step waits for this kernel): a thread per four columns, the row read
     // in one pass; many rows: fewer threads per row, more rows per SM
@@ -501,7 +509,7 @@ SOMI_API int somi_add_layernorm(float* residual, const void* delta, int delta_dt
                    delta_split_stride, static_cast<const TG*>(gate), gate_stride, gate_splits,   \
                    gate_split_stride, weight,                                                    \
                    weight_dtype, eps, static_cast<TO*>(out), rows, H, write_back, rms, vec4,     \
-                   extra);                                                                       \
+                   extra, bias);                                                                       \
     } while (0)
     // the output is of the compute dtype; the delta and the gate are that or float32 partial sums
     if (out_dtype == SOMI_F32) {

@@ -131,12 +131,10 @@ __global__ void unary_act_kernel(const T* __restrict__ x, T* __restrict__ out, l
         out[i] = from_float<T>(unary_act(to_float(x[i]), kind));
 }
 
-// The experts' activation over a product whose columns alternate gate_j, up_j:
-// out[r, j] = g * sigmoid(alpha * g) * (u + shift), g = min(gate, limit), u = clamp(up, -limit, limit)
-// (limit = infinity, alpha = 1, shift = 0: silu(gate) * up).
+// A gated activation over a product whose columns alternate gate_j, up_j: out[r, j] = glu(gate, up).
 template <typename T>
 __global__ void clamped_gate_up_kernel(const T* __restrict__ gu, T* __restrict__ out, int ff,
-                                       long long n, float limit, float alpha, float shift) {
+                                       long long n, GluForm form) {
     pdl_launch_dependents();
     pdl_wait();
     if (sizeof(T) == 2 && (n & 3) == 0 && ((reinterpret_cast<uintptr_t>(gu) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
@@ -150,9 +148,7 @@ __global__ void clamped_gate_up_kernel(const T* __restrict__ gu, T* __restrict__
             float y[4];
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const float g = fminf(__low2float(h[e]), limit);
-                const float u = fminf(fmaxf(__high2float(h[e]), -limit), limit);
-                y[e] = g / (1.0f + expf(-alpha * g)) * (u + shift);
+                y[e] = glu(__low2float(h[e]), __high2float(h[e]), form);
             }
             const __nv_bfloat162 y01 = __floats2bfloat162_rn(y[0], y[1]), y23 = __floats2bfloat162_rn(y[2], y[3]);
             uint2 packed;
@@ -164,9 +160,7 @@ __global__ void clamped_gate_up_kernel(const T* __restrict__ gu, T* __restrict__
     }
     for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n;
          i += static_cast<long long>(gridDim.x) * blockDim.x) {
-        const float g = fminf(to_float(gu[2 * i]), limit);
-        const float u = fminf(fmaxf(to_float(gu[2 * i + 1]), -limit), limit);
-        out[i] = from_float<T>(g / (1.0f + expf(-alpha * g)) * (u + shift));
+        out[i] = from_float<T>(glu(to_float(gu[2 * i]), to_float(gu[2 * i + 1]), form));
     }
 }
 
@@ -183,7 +177,7 @@ __global__ void __launch_bounds__(kGemvWarps * 32)
 moe_gemv_kernel(const __nv_bfloat16* __restrict__ A, long long a_stride, int a_div,
                 const __nv_bfloat16* __restrict__ W, const int* __restrict__ ids,
                 const int* __restrict__ table, int top, int E, void* __restrict__ out, int N, int K,
-                float limit, float alpha, float shift, int act) {
+                GluForm form, int act) {
     extern __shared__ float xs[];                          // [K]
     pdl_launch_dependents();
     pdl_wait();
@@ -220,10 +214,8 @@ moe_gemv_kernel(const __nv_bfloat16* __restrict__ A, long long a_stride, int a_d
         a1 = warp_sum(a1);
         if (lane == 0) {
             if (MODE == 1) {
-                const float g = fminf(a0, limit);
-                const float u = fminf(fmaxf(a1, -limit), limit);
                 static_cast<__nv_bfloat16*>(out)[static_cast<size_t>(entry) * (N / 2) + row / 2] =
-                    __float2bfloat16_rn(g / (1.0f + expf(-alpha * g)) * (u + shift));
+                    __float2bfloat16_rn(glu(a0, a1, form));
             } else if (MODE == 2) {
                 __nv_bfloat16* o = static_cast<__nv_bfloat16*>(out) + static_cast<size_t>(entry) * N;
                 o[row] = __float2bfloat16_rn(unary_act(a0, act));
@@ -238,8 +230,7 @@ moe_gemv_kernel(const __nv_bfloat16* __restrict__ A, long long a_stride, int a_d
 }
 
 // MODE 0: out (TO) rows at `scatter` positions (or the sorted position itself), N columns.
-// MODE 1: W's rows alternate gate_j, up_j; g = min(gate, limit), u = clamp(up, -limit, limit);
-//         out[pos, j] = g * sigmoid(alpha * g) * (u + shift), N / 2 columns.
+// MODE 1: W's rows alternate gate_j, up_j; out[pos, j] = glu(gate, up), N / 2 columns.
 // MODE 2: out[pos, c] = act(product), N columns (an expert without a gate).
 template <typename T, typename TO, int MODE>
 __global__ void __launch_bounds__(kMoeThreads)
@@ -247,8 +238,8 @@ grouped_gemm_kernel(const T* __restrict__ A, long long a_stride, const int* __re
                     int gather_div, const T* __restrict__ W, const int* __restrict__ offsets,
                     const int* __restrict__ tile_expert, const int* __restrict__ tile_row0,
                     const int* __restrict__ n_tiles, int n_rows_single, TO* __restrict__ out,
-                    long long out_stride, const int* __restrict__ scatter, int N, int K, float limit,
-                    float alpha, float shift, int act) {
+                    long long out_stride, const int* __restrict__ scatter, int N, int K, GluForm form,
+                    int act) {
     __shared__ float As[kMoeBK][kMoeBM + 1];
     __shared__ float Ws[kMoeBK][kMoeBN + 1];
     __shared__ int rows_s[kMoeBM];
@@ -332,10 +323,8 @@ grouped_gemm_kernel(const T* __restrict__ A, long long a_stride, const int* __re
             for (int j = 0; j < 4; j += 2) {
                 const int c = col0 + tx * 4 + j;       // even: a gate row; c + 1 its up row
                 if (c + 1 < N) {
-                    const float g = fminf(acc[i][j], limit);
-                    const float u = fminf(fmaxf(acc[i][j + 1], -limit), limit);
-                    const float y = g / (1.0f + expf(-alpha * g)) * (u + shift);
-                    out[static_cast<size_t>(pos) * out_stride + c / 2] = from_float<TO>(y);
+                    out[static_cast<size_t>(pos) * out_stride + c / 2] =
+                        from_float<TO>(glu(acc[i][j], acc[i][j + 1], form));
                 }
             }
         }
@@ -398,12 +387,12 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restri
 // Equal values go to the lower index.  With `over_chosen` the choice is made on the logits
 // themselves (no correction, no groups) and the weights are the softmax over the chosen logits only.
 // `sigmoid`: s = sigmoid(logits) instead of the softmax; `group_best` 2: a group's score is the sum of
-// its two largest choices (of its only one where it has one member).
+// its two largest choices (of its only one where it has one member).  All weights are multiplied by `factor`.
 __global__ void moe_router_select_kernel(const float* __restrict__ logits, long long l_stride,
                                          const float* __restrict__ correction, int n, int count,
                                          int keep, int top, int* __restrict__ chosen,
                                          float* __restrict__ weight, int T, int over_chosen,
-                                         int sigmoid, int group_best) {
+                                         int sigmoid, int group_best, float factor) {
     extern __shared__ float rs[];            // per warp: s [n], choice [n], group score [count]
     pdl_launch_dependents();
     pdl_wait();
@@ -478,7 +467,7 @@ __global__ void moe_router_select_kernel(const float* __restrict__ logits, long 
         if (arg == 0x7fffffff) arg = 0;
         if (lane == 0) {
             chosen[static_cast<size_t>(t) * top + k] = arg;
-            weight[static_cast<size_t>(t) * top + k] = sv[arg];
+            weight[static_cast<size_t>(t) * top + k] = sv[arg] * factor;
             cv[arg] = NAN;                    // taken: not chosen again
         }
         __syncwarp();
@@ -489,26 +478,33 @@ __global__ void moe_router_select_kernel(const float* __restrict__ logits, long 
         const float zmax = z[c[0]];
         float den = 0.f;
         for (int k = 0; k < top; ++k) { w[k] = expf(z[c[k]] - zmax); den += w[k]; }
-        for (int k = 0; k < top; ++k) w[k] /= den;
+        for (int k = 0; k < top; ++k) w[k] = w[k] / den * factor;
     }
 }
 
 // out[t, c] = sum_k weight[t, k] * (table[t, k] < E ? y[row(t * top + k), c] : x[t, c]); float32.
 // row(e) = place[e] where the rows of y are in the grouped order, else e.  The sum runs over k in
 // ascending order.
+// `side` (or null): the result of an expert that every token passes, [side_splits] partial sums (TS) that
+// lie `side_stride` elements apart and are added in order; with `side_gate` (float32, tokens
+// `gate_stride` apart) it joins the sum times sigmoid(side_gate[t]).
 // A CTA per token (its entries of table, weight and place are read once by every warp); a thread
 // four neighbouring columns where the rows allow it (`vec`), else one.
-template <typename TY, typename TX>
+template <typename TY, typename TX, typename TS>
 __global__ void moe_combine_weighted_kernel(const TY* __restrict__ y, const int* __restrict__ place,
                                             const int* __restrict__ table,
                                             const float* __restrict__ weight, const TX* __restrict__ x,
-                                            int E, int top, int H, int T, int vec, float* __restrict__ out) {
+                                            int E, int top, int H, int T, int vec,
+                                            const TS* __restrict__ side, int side_splits,
+                                            long long side_stride, const float* __restrict__ side_gate,
+                                            long long gate_stride, float* __restrict__ out) {
     pdl_launch_dependents();
     pdl_wait();
     for (int t = blockIdx.x; t < T; t += gridDim.x) {
         const long long e0 = static_cast<long long>(t) * top;
         const TX* xr = x + static_cast<size_t>(t) * H;
         float* o = out + static_cast<size_t>(t) * H;
+        const float sg = side_gate != nullptr ? 1.0f / (1.0f + expf(-side_gate[t * gate_stride])) : 1.0f;
         if (vec) {
             for (int c = 4 * threadIdx.x; c < H; c += 4 * blockDim.x) {
                 F4 s{{0.f, 0.f, 0.f, 0.f}};
@@ -521,6 +517,16 @@ __global__ void moe_combine_weighted_kernel(const TY* __restrict__ y, const int*
 #pragma unroll
                     for (int j = 0; j < 4; ++j) s.v[j] = fmaf(w, v.v[j], s.v[j]);
                 }
+                if (side != nullptr) {
+                    F4 d = load4(side + static_cast<size_t>(t) * H + c);
+                    for (int sp = 1; sp < side_splits; ++sp) {
+                        const F4 v = load4(side + sp * side_stride + static_cast<size_t>(t) * H + c);
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) d.v[j] += v.v[j];
+                    }
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) s.v[j] = fmaf(sg, d.v[j], s.v[j]);
+                }
                 store4(o + c, s);
             }
         } else {
@@ -532,6 +538,11 @@ __global__ void moe_combine_weighted_kernel(const TY* __restrict__ y, const int*
                         ? to_float(y[static_cast<size_t>(place != nullptr ? place[e0 + k] : e0 + k) * H + c])
                         : to_float(xr[c]);
                     s = fmaf(weight[e0 + k], v, s);
+                }
+                if (side != nullptr) {
+                    float d = to_float(side[static_cast<size_t>(t) * H + c]);
+                    for (int sp = 1; sp < side_splits; ++sp) d += to_float(side[sp * side_stride + static_cast<size_t>(t) * H + c]);
+                    s = fmaf(sg, d, s);
                 }
                 o[c] = s;
             }
@@ -579,17 +590,18 @@ SOMI_API int somi_moe_gather_rows(const void* a, int dtype, long long a_stride, 
 }
 
 SOMI_API int somi_clamped_gate_up(const void* gu, void* out, int dtype, long long rows, int ff,
-                                  float limit, float alpha, float shift, cudaStream_t stream) {
+                                  float limit, float alpha, float shift, float cubic, cudaStream_t stream) {
     const long long n = rows * ff;
     if (n <= 0) return 0;
     const int blocks = static_cast<int>(((n + 255) / 256) < 148LL * 16 ? ((n + 255) / 256) : 148LL * 16);
     if (dtype == SOMI_F32)
         launch_pdl(clamped_gate_up_kernel<float>, dim3(blocks), dim3(256), 0, stream,
-                   static_cast<const float*>(gu), static_cast<float*>(out), ff, n, limit, alpha, shift);
+                   static_cast<const float*>(gu), static_cast<float*>(out), ff, n,
+                   GluForm{limit, alpha, shift, cubic});
     else
         launch_pdl(clamped_gate_up_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream,
                    static_cast<const __nv_bfloat16*>(gu), static_cast<__nv_bfloat16*>(out), ff, n,
-                   limit, alpha, shift);
+                   GluForm{limit, alpha, shift, cubic});
     return launch_status();
 }
 
@@ -611,7 +623,8 @@ SOMI_API int somi_unary_act(const void* x, void* out, int dtype, long long n, in
 // float32 rows [entries, N].  Row e of A is a[e / a_div].
 SOMI_API int somi_moe_gemv(const void* A, long long a_stride, int a_div, const void* W, const int* ids,
                            const int* table, int top, int E, int n_entries, void* out, int N, int K,
-                           int mode, float limit, float alpha, float shift, int act, cudaStream_t stream) {
+                           int mode, float limit, float alpha, float shift, float cubic, int act,
+                           cudaStream_t stream) {
     if (n_entries <= 0) return 0;
     if (K <= 0 || (K & 7) || N <= 0 || (mode == 1 && (N & 1)) || K > 40 * 1024 ||
         (reinterpret_cast<uintptr_t>(W) & 15))
@@ -623,19 +636,22 @@ SOMI_API int somi_moe_gemv(const void* A, long long a_stride, int a_div, const v
             cudaFuncSetAttribute(moe_gemv_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         launch_pdl(moe_gemv_kernel<1>, grid, dim3(kGemvWarps * 32), smem, stream,
                    static_cast<const __nv_bfloat16*>(A), a_stride, a_div,
-                   static_cast<const __nv_bfloat16*>(W), ids, table, top, E, out, N, K, limit, alpha, shift, act);
+                   static_cast<const __nv_bfloat16*>(W), ids, table, top, E, out, N, K,
+                   GluForm{limit, alpha, shift, cubic}, act);
     } else if (mode == 2) {
         if (smem > 48 * 1024)
             cudaFuncSetAttribute(moe_gemv_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         launch_pdl(moe_gemv_kernel<2>, grid, dim3(kGemvWarps * 32), smem, stream,
                    static_cast<const __nv_bfloat16*>(A), a_stride, a_div,
-                   static_cast<const __nv_bfloat16*>(W), ids, table, top, E, out, N, K, limit, alpha, shift, act);
+                   static_cast<const __nv_bfloat16*>(W), ids, table, top, E, out, N, K,
+                   GluForm{limit, alpha, shift, cubic}, act);
     } else {
         if (smem > 48 * 1024)
             cudaFuncSetAttribute(moe_gemv_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         launch_pdl(moe_gemv_kernel<0>, grid, dim3(kGemvWarps * 32), smem, stream,
                    static_cast<const __nv_bfloat16*>(A), a_stride, a_div,
-                   static_cast<const __nv_bfloat16*>(W), ids, table, top, E, out, N, K, limit, alpha, shift, act);
+                   static_cast<const __nv_bfloat16*>(W), ids, table, top, E, out, N, K,
+                   GluForm{limit, alpha, shift, cubic}, act);
     }
     return launch_status();
 }
@@ -647,7 +663,8 @@ SOMI_API int somi_grouped_gemm(const void* A, int dtype, long long a_stride, int
                                int use_gather, const void* W, const int* work, int E, int n_entries,
                                int max_tiles, int n_rows, void* out, int out_f32,
                                long long out_stride, int use_scatter, int N, int K, int mode,
-                               float limit, float alpha, float shift, int act, cudaStream_t stream) {
+                               float limit, float alpha, float shift, float cubic, int act,
+                           cudaStream_t stream) {
     if (N <= 0 || K <= 0) return SOMI_ERR_UNSUPPORTED;
     const int* offsets = nullptr; const int* sorted = nullptr; const int* tile_expert = nullptr;
     const int* tile_row0 = nullptr; const int* n_tiles = nullptr;
@@ -671,7 +688,7 @@ SOMI_API int somi_grouped_gemm(const void* A, int dtype, long long a_stride, int
     launch_pdl(grouped_gemm_kernel<TT, TO, MODE>, grid, dim3(kMoeThreads), 0, stream,            \
                static_cast<const TT*>(A), a_stride, gather, gather_div, static_cast<const TT*>(W), \
                offsets, tile_expert, tile_row0, n_tiles, n_rows, static_cast<TO*>(out), out_stride, \
-               scatter, N, K, limit, alpha, shift, act)
+               scatter, N, K, GluForm{limit, alpha, shift, cubic}, act)
     if (dtype == SOMI_F32) {
         if (mode == 1) SOMI_LAUNCH_GG(float, float, 1);
         else if (mode == 2) SOMI_LAUNCH_GG(float, float, 2);
@@ -704,7 +721,7 @@ SOMI_API int somi_moe_combine(const void* y, int y_dtype, const int* place, cons
 SOMI_API int somi_moe_router_select(const float* logits, long long l_stride, const float* correction,
                                     int T, int n, int count, int keep, int top, int* chosen,
                                     float* weight, int over_chosen, int sigmoid, int group_best,
-                                    cudaStream_t stream) {
+                                    float factor, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (n <= 0 || n > 4096 || top <= 0 || top > n || (count > 1 && (n % count || keep <= 0 || keep > count)))
         return SOMI_ERR_UNSUPPORTED;
@@ -716,25 +733,42 @@ SOMI_API int somi_moe_router_select(const float* logits, long long l_stride, con
         cudaFuncSetAttribute(moe_router_select_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_pdl(moe_router_select_kernel, dim3((T + warps - 1) / warps), dim3(32 * warps), smem, stream,
                logits, l_stride, correction, n, count, keep, top, chosen, weight, T, over_chosen, sigmoid,
-               group_best);
+               group_best, factor);
     return launch_status();
 }
 
+// `side`: null, or side_splits partial sums [T, H] of side_dtype (more than one: float32); `side_gate`: null,
+// or float32 logits, one per token, gate_stride apart.
 SOMI_API int somi_moe_combine_weighted(const void* y, int y_dtype, const int* place, const int* table,
                                        const float* weight, const void* x, int x_dtype, int E, int top,
-                                       int T, int H, float* out, cudaStream_t stream) {
+                                       int T, int H, const void* side, int side_dtype, int side_splits,
+                                       long long side_stride, const float* side_gate,
+                                       long long gate_stride, float* out, cudaStream_t stream) {
     if (T <= 0 || H <= 0) return 0;
-    const int vec = (H % 4 == 0 && ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(x) |
-                                     reinterpret_cast<uintptr_t>(out)) & 15) == 0) ? 1 : 0;
+    if (side != nullptr && (side_splits < 1 || (side_splits > 1 && side_dtype != SOMI_F32))) return SOMI_ERR_UNSUPPORTED;
+    const int vec = (H % 4 == 0 && side_stride % 4 == 0 &&
+                     ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(x) |
+                       reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(side)) & 15) == 0) ? 1 : 0;
     const int threads = min(256, max(32, ((H / (vec ? 4 : 1) + 31) / 32) * 32));
     const int blocks = min(T, 148 * 32);
-#define SOMI_LAUNCH_CW(TY, TX)                                                                    \
-    launch_pdl(moe_combine_weighted_kernel<TY, TX>, dim3(blocks), dim3(threads), 0, stream,       \
-               static_cast<const TY*>(y), place, table, weight, static_cast<const TX*>(x), E, top, H, T, vec, out)
-    if (y_dtype == SOMI_F32 && x_dtype == SOMI_F32) SOMI_LAUNCH_CW(float, float);
-    else if (y_dtype == SOMI_F32) SOMI_LAUNCH_CW(float, __nv_bfloat16);
-    else if (x_dtype == SOMI_F32) SOMI_LAUNCH_CW(__nv_bfloat16, float);
-    else SOMI_LAUNCH_CW(__nv_bfloat16, __nv_bfloat16);
+#define SOMI_LAUNCH_CW(TY, TX, TS)                                                                \
+    launch_pdl(moe_combine_weighted_kernel<TY, TX, TS>, dim3(blocks), dim3(threads), 0, stream,   \
+               static_cast<const TY*>(y), place, table, weight, static_cast<const TX*>(x), E, top, H, T, vec, \
+               static_cast<const TS*>(side), side_splits, side_stride, side_gate, gate_stride, out)
+    const bool side_f32 = side == nullptr || side_dtype == SOMI_F32;
+    if (y_dtype == SOMI_F32 && x_dtype == SOMI_F32) {
+        if (!side_f32) return SOMI_ERR_UNSUPPORTED;
+        SOMI_LAUNCH_CW(float, float, float);
+    } else if (y_dtype == SOMI_F32) {
+        if (side_f32) SOMI_LAUNCH_CW(float, __nv_bfloat16, float);
+        else SOMI_LAUNCH_CW(float, __nv_bfloat16, __nv_bfloat16);
+    } else if (x_dtype == SOMI_F32) {
+        if (!side_f32) return SOMI_ERR_UNSUPPORTED;
+        SOMI_LAUNCH_CW(__nv_bfloat16, float, float);
+    } else {
+        if (side_f32) SOMI_LAUNCH_CW(__nv_bfloat16, __nv_bfloat16, float);
+        else SOMI_LAUNCH_CW(__nv_bfloat16, __nv_bfloat16, __nv_bfloat16);
+    }
 #undef SOMI_LAUNCH_CW
     return launch_status();
 }

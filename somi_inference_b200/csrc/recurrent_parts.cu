@@ -141,17 +141,21 @@ __global__ void add_scaled_rmsnorm_kernel(float* __restrict__ residual, const vo
 // then entry i < rot/2 and entry i + rot/2 of the token at position p turn by p * inv_freq[i]
 // (the angle is formed and reduced in float64, its sine and cosine are float32 and are both
 // multiplied by `magnitude`, 1 for a plain rotation); entries from `rot` on pass.  Queries are written back in place; keys and values go to their cache slots.
+// `maps` neighbouring key heads lie side by side in one cache row of maps * hd elements and share
+// one value head (there are nkv / maps of these).
 // One warp per head; the normed head passes through shared memory so that a lane finds its partner.
+// Sines and cosines are made once per token.
 template <typename T>
 __global__ void headnorm_rotary_store_kernel(T* __restrict__ qkv, long long stride,
                                              const int* __restrict__ positions,
                                              const double* __restrict__ inv_freq, int nq, int nkv,
                                              int hd, int vd, int rot, const void* __restrict__ q_w,
                                              const void* __restrict__ k_w, int w_dtype, float eps,
-                                             float magnitude,
+                                             float magnitude, int maps,
                                              const int* __restrict__ slot_map, T* __restrict__ kcache,
                                              T* __restrict__ vcache, int page_size) {
-    extern __shared__ float heads_s[];                 // [warps][hd]
+    extern __shared__ float2 cs_s[];                   // [rot / 2] cosine, sine; then [warps][hd]
+    float* heads_s = reinterpret_cast<float*>(cs_s + (rot >> 1));
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -161,7 +165,12 @@ __global__ void headnorm_rotary_store_kernel(T* __restrict__ qkv, long long stri
     const int slot = slot_map != nullptr ? slot_map[t] : -1;
     const size_t page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot % page_size : 0;
     float* mine = heads_s + warp * hd;
-    const int half = rot >> 1;
+    const int half = rot >> 1, nv = nkv / maps;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        const float2 cs = turn_by(pos, inv_freq[i]);
+        cs_s[i] = make_float2(cs.x * magnitude, cs.y * magnitude);
+    }
+    __syncthreads();
     for (int head = blockIdx.y * nwarps + warp; head < nq + nkv; head += nwarps * gridDim.y) {
         T* x = row + static_cast<size_t>(head) * hd;
         const void* w = head < nq ? q_w : k_w;
@@ -179,19 +188,14 @@ __global__ void headnorm_rotary_store_kernel(T* __restrict__ qkv, long long stri
         __syncwarp();
         T* dst = nullptr;
         if (head < nq) dst = x;
-        else if (slot >= 0) dst = kcache + ((page * nkv + (head - nq)) * page_size + off) * hd;
+        else if (slot >= 0)
+            dst = kcache + (((page * nv + (head - nq) / maps) * page_size + off) * maps + (head - nq) % maps) * hd;
         if (dst != nullptr) {
             for (int e = lane; e < hd; e += 32) {
                 float v = mine[e];
                 if (e < rot) {
-                    const int i = e < half ? e : e - half;
-                    double angle = pos * inv_freq[i];
-                    angle -= 6.283185307179586476925286766559 * rint(angle * 0.15915494309189533576888376337251);
-                    float sn, cs;
-                    sincosf(static_cast<float>(angle), &sn, &cs);
-                    sn *= magnitude;
-                    cs *= magnitude;
-                    v = e < half ? fmaf(v, cs, -(mine[e + half] * sn)) : fmaf(v, cs, mine[e - half] * sn);
+                    const float2 cs = cs_s[e < half ? e : e - half];
+                    v = e < half ? fmaf(v, cs.x, -(mine[e + half] * cs.y)) : fmaf(v, cs.x, mine[e - half] * cs.y);
                 }
                 dst[e] = from_float<T>(v);
             }
@@ -200,8 +204,8 @@ __global__ void headnorm_rotary_store_kernel(T* __restrict__ qkv, long long stri
     }
     if (slot >= 0 && blockIdx.y == 0) {
         const T* vrow = row + static_cast<size_t>(nq + nkv) * hd;
-        for (int g = 0; g < nkv; ++g) {
-            T* dst = vcache + ((page * nkv + g) * page_size + off) * vd;
+        for (int g = 0; g < nv; ++g) {
+            T* dst = vcache + ((page * nv + g) * page_size + off) * vd;
             for (int e = threadIdx.x; e < vd; e += blockDim.x) dst[e] = vrow[static_cast<size_t>(g) * vd + e];
         }
     }
@@ -804,23 +808,24 @@ SOMI_API int somi_add_scaled_rmsnorm(float* residual, const void* a, int a_dtype
 SOMI_API int somi_headnorm_rotary_store(void* qkv, int dtype, long long stride, const int* positions,
                                         const double* inv_freq, int T, int nq, int nkv, int hd, int vd,
                                         int rot, const void* q_w, const void* k_w, int w_dtype,
-                                        float eps, float magnitude, const int* slot_map, void* kcache,
-                                        void* vcache, int page_size, cudaStream_t stream) {
+                                        float eps, float magnitude, int maps, const int* slot_map,
+                                        void* kcache, void* vcache, int page_size, cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (hd <= 0 || hd > 1024 || vd <= 0 || rot < 0 || rot > hd || (rot & 1) || nq <= 0 || nkv <= 0)
+    if (hd <= 0 || hd > 1024 || vd <= 0 || rot < 0 || rot > hd || (rot & 1) || nq <= 0 || nkv <= 0 ||
+        maps <= 0 || nkv % maps)
         return SOMI_ERR_UNSUPPORTED;
     const int warps = min(8, nq + nkv);
     const dim3 grid(T, T <= 256 ? (nq + nkv + 7) / 8 : 1);
-    const size_t smem = sizeof(float) * warps * hd;
+    const size_t smem = sizeof(float) * warps * hd + sizeof(float2) * (rot >> 1);
     if (dtype == SOMI_F32)
         launch_pdl(headnorm_rotary_store_kernel<float>, grid, dim3(32 * warps), smem, stream,
                    static_cast<float*>(qkv), stride, positions, inv_freq, nq, nkv, hd, vd, rot, q_w,
-                   k_w, w_dtype, eps, magnitude, slot_map, static_cast<float*>(kcache),
+                   k_w, w_dtype, eps, magnitude, maps, slot_map, static_cast<float*>(kcache),
                    static_cast<float*>(vcache), page_size);
     else
         launch_pdl(headnorm_rotary_store_kernel<__nv_bfloat16>, grid, dim3(32 * warps), smem, stream,
                    static_cast<__nv_bfloat16*>(qkv), stride, positions, inv_freq, nq, nkv, hd, vd,
-                   rot, q_w, k_w, w_dtype, eps, magnitude, slot_map, static_cast<__nv_bfloat16*>(kcache),
+                   rot, q_w, k_w, w_dtype, eps, magnitude, maps, slot_map, static_cast<__nv_bfloat16*>(kcache),
                    static_cast<__nv_bfloat16*>(vcache), page_size);
     return launch_status();
 }

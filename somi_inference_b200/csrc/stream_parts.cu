@@ -429,8 +429,8 @@ __global__ void __launch_bounds__(256)
 latent_rotary_store_kernel(const T* __restrict__ x, long long stride, int q_at, int H, int qd, int rot,
                            int c_at, int rank, int neighbours, const int* __restrict__ positions,
                            const double* __restrict__ inv_freq, const void* __restrict__ weight,
-                           int w_dtype, float eps, const int* __restrict__ slot_map, T* __restrict__ cache,
-                           T* __restrict__ qa, int n_tokens, int vec2) {
+                           int w_dtype, float eps, float magnitude, const int* __restrict__ slot_map,
+                           T* __restrict__ cache, T* __restrict__ qa, int n_tokens, int vec2) {
     extern __shared__ float2 cs_s[];                       // [rot / 2]
     __shared__ float scratch[33];
     pdl_launch_dependents();
@@ -439,7 +439,10 @@ latent_rotary_store_kernel(const T* __restrict__ x, long long stride, int q_at, 
     const T* row = x + static_cast<size_t>(t) * stride;
     const int half = rot >> 1, W = rank + rot;
     const double pos = static_cast<double>(positions[t]);
-    for (int i = tid; i < half; i += nthr) cs_s[i] = turn_by(pos, inv_freq[i]);
+    for (int i = tid; i < half; i += nthr) {
+        const float2 cs = turn_by(pos, inv_freq[i]);
+        cs_s[i] = make_float2(cs.x * magnitude, cs.y * magnitude);
+    }
     float ss = 0.f;
     if (vec2) {
         for (int e = 2 * tid; e < rank; e += 2 * nthr) {
@@ -467,6 +470,21 @@ latent_rotary_store_kernel(const T* __restrict__ x, long long stride, int q_at, 
             for (int e = tid; e < rank; e += nthr)
                 dst[e] = from_float<T>(to_float(row[c_at + e]) * inv * load_as_float(weight, w_dtype, e));
         }
+    }
+    if (vec2 && !neighbours) {
+        // two neighbouring pairs (j, j + half), (j + 1, j + 1 + half) at once
+        for (int it = tid; it < (H + 1) * (half >> 1); it += nthr) {
+            const int h = it / (half >> 1), j = 2 * (it - h * (half >> 1));
+            const T* src = h < H ? row + q_at + static_cast<size_t>(h) * (qd + rot) + qd : row + c_at + rank;
+            T* dst;
+            if (h < H) dst = qa + (static_cast<size_t>(h) * n_tokens + t) * W + rank;
+            else if (slot_map != nullptr) dst = cache + static_cast<size_t>(slot_map[t]) * W + rank;
+            else continue;
+            const float2 c0 = cs_s[j], c1 = cs_s[j + 1], u = load2(src + j), v = load2(src + j + half);
+            store2(dst + j, fmaf(u.x, c0.x, -(v.x * c0.y)), fmaf(u.y, c1.x, -(v.y * c1.y)));
+            store2(dst + j + half, fmaf(v.x, c0.x, u.x * c0.y), fmaf(v.y, c1.x, u.y * c1.y));
+        }
+        return;
     }
     for (int it = tid; it < (H + 1) * half; it += nthr) {
         const int h = it / half, j = it - h * half;
@@ -595,18 +613,18 @@ SOMI_API int somi_turn_back(void* x, int dtype, const float* turn, long long row
 SOMI_API int somi_latent_rotary_store(const void* x, int dtype, long long stride, int q_at, int H,
                                       int qd, int rot, int c_at, int rank, int neighbours,
                                       const int* positions, const double* inv_freq, const void* weight,
-                                      int w_dtype, float eps, const int* slot_map, void* cache,
-                                      void* qa, int T, cudaStream_t stream) {
+                                      int w_dtype, float eps, float magnitude, const int* slot_map,
+                                      void* cache, void* qa, int T, cudaStream_t stream) {
     if (T <= 0) return 0;
     if (H <= 0 || qd < 0 || rot < 0 || (rot & 1) || rot > 4096 || rank <= 0) return SOMI_ERR_UNSUPPORTED;
     const size_t smem = sizeof(float2) * (rot / 2 + 1);
-    const int vec2 = neighbours && ((q_at | qd | c_at | rank) & 1) == 0 && (stride & 1) == 0 && aligned16(x) &&
+    const int vec2 = (neighbours || (rot & 3) == 0) && ((q_at | qd | c_at | rank) & 1) == 0 && (stride & 1) == 0 && aligned16(x) &&
                      aligned16(cache) && aligned16(qa);
 #define SOMI_LAUNCH_LRS(TT)                                                                        \
     launch_pdl(latent_rotary_store_kernel<TT>, dim3(T), dim3(256), smem, stream,                   \
                static_cast<const TT*>(x), stride, q_at, H, qd, rot, c_at, rank, neighbours,        \
-               positions, inv_freq, weight, w_dtype, eps, slot_map, static_cast<TT*>(cache),       \
-               static_cast<TT*>(qa), T, vec2)
+               positions, inv_freq, weight, w_dtype, eps, magnitude, slot_map,                     \
+               static_cast<TT*>(cache), static_cast<TT*>(qa), T, vec2)
     if (dtype == SOMI_F32) SOMI_LAUNCH_LRS(float);
     else SOMI_LAUNCH_LRS(__nv_bfloat16);
 #undef SOMI_LAUNCH_LRS

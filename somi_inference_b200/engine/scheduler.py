@@ -126,7 +126,8 @@ class Scheduler:
         that keeps all keys: ceil((prompt + max_new - 1) / page_size), as
         continuous_batching.py:64-67.  A group with a window of w keeps the pages between the
         oldest key a query still reads and the end of the portion being written: at most
-        ceil((w + portion) / page_size) + 1, whatever the length."""
+        ceil((w + portion) / page_size) + 1, whatever the length, and the pages of the first
+        positions where these stay readable."""
         full = self._pages_for(len(req.prompt_tokens) + req.max_new_tokens - 1)
         out = []
         for g in self.cache.groups:
@@ -134,7 +135,7 @@ class Scheduler:
             if w is None:
                 out.append(full)
             else:
-                out.append(min(full, self._pages_for(w + self.chunk_size) + 1))
+                out.append(min(full, self._pages_for(w + self.chunk_size) + 1 + g.kept))
         return out
 
     def add_request(self, req: Request) -> None:

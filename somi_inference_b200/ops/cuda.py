@@ -268,7 +268,7 @@ class CudaOps:
 
     @staticmethod
     def _attention_work(batch, first: int, last: int, nq: int, nkv: int, hd: int, elt: int,
-                        window: int) -> tuple[float, float]:
+                        window: int, keep: int = 0) -> tuple[float, float]:
         """Bytes and flops of attention for requests [first, last) of the batch: every key and
         value of a request's context once, queries in and outputs out; two products per
         (query, key) pair that the mask leaves."""
@@ -283,8 +283,10 @@ class CudaOps:
                 pairs = sum((c + i) % n + 1 for i in range(q)) if q < 4096 else min(pairs, q * n // 2)
                 kv = min(kv, (c % n) + q)
             elif window:
-                pairs = sum(min(c + i + 1, window) for i in range(q)) if q < 4096 else min(pairs, q * window)
-                kv = min(kv, window + q - 1)
+                # (and the first `keep` keys)
+                pairs = (sum(min(c + i + 1, window + keep) for i in range(q)) if q < 4096
+                         else min(pairs, q * (window + keep)))
+                kv = min(kv, window + keep + q - 1)
             moved += 2 * kv * nkv * hd * elt + 2 * q * nq * hd * elt
             flops += 4.0 * nq * hd * pairs
         return moved, flops
@@ -459,7 +461,7 @@ class CudaOps:
                 ctypes.c_int(max(win, 0)), ctypes.c_int(chunk), _ptr(gate),
                 ctypes.c_longlong(gate.stride(0) if gate is not None else 0),
                 ctypes.c_int(1 if gate_per_head else 0), ctypes.c_float(cap), _ptr(sinks),
-                _ptr(out), self._stream())
+                ctypes.c_int(0), ctypes.c_int(1), ctypes.c_int(0), _ptr(out), self._stream())
             self._done(rc, "paged_attention")
             if trace.active():
                 first = batch.num_prefill_requests if tensor_core_prefill else 0
@@ -520,15 +522,119 @@ class CudaOps:
             first = 0 if tensor_core_prefill else batch.num_prefill_tokens
             last = batch.num_tokens if split else batch.num_prefill_tokens
             if gate_per_head:
-                rc = self.lib.somi_head_gate_mul(
-                    _ptr(out[first:last]), _ptr(gate[first:last]), _code(out),
-                    ctypes.c_longlong(gate.stride(0)), ctypes.c_longlong(last - first),
-                    ctypes.c_int(nq), ctypes.c_int(vd), self._stream())
-                self._done(rc, "head_gate_mul")
-                if trace.active():
-                    trace.note("head_gate_mul", 2 * (last - first) * nq * vd * out.element_size())
+                self.head_gate_mul(out[first:last], gate[first:last], nq)
             else:
                 self.sigmoid_gate_mul(out[first:last], gate[first:last])
+
+    def two_map_attention(self, qkv, kcache, vcache, batch, group, nq, nkv, d, vd, scale, window, keep,
+                          factor: float, eps: float, gain: float, gate, out, storage=None) -> None:
+        """Attention in two maps of every token of the step over the cache (keys and values already
+        stored).  Rows of `qkv` begin with nq heads of two queries of `d` elements; a key row of the
+        cache ([pages, nkv, page, 2 d]) holds two keys, a value row `vd` elements.  Query n of a head
+        meets key n, with scores q.k * scale over the keys at most `window` - 1 back (None: all
+        earlier ones) and those at positions below `keep`; with a1, a2 the two outputs and
+        e = a1 - factor * a2, the head's output is e / sqrt(mean(e^2) + eps) * gain, times
+        sigmoid(gate[t, head]) (`gate`: logits [T, nq] whose rows may lie further apart, or None).
+
+        bfloat16 with 2 d = vd = 64 or 128: prompt portions run the two-tile tcgen05 kernel, whose
+        two tiles are then the two maps, single tokens the split-KV kernels fed by TMA with a merge
+        that takes the difference.  Otherwise the kernel for any size leaves both maps in float32
+        and a kernel behind it takes the difference."""
+        _check(qkv, kcache, vcache, out, group.block_table)
+        assert kcache.dtype == vcache.dtype == qkv.dtype == out.dtype
+        assert kcache.shape[1] == vcache.shape[1] == nkv and kcache.shape[3] == 2 * d and vcache.shape[3] == vd
+        assert tuple(out.shape) == (batch.num_tokens, nq * vd)
+        if gate is not None and not (gate.is_cuda and gate.dtype == out.dtype and gate.stride(1) == 1
+                                     and tuple(gate.shape) == (out.shape[0], nq)):
+            raise KernelError("a gate per head is [T, heads] of the output's dtype with contiguous rows")
+        page_size = kcache.shape[2]
+        win, keep = int(window) if window else 0, int(keep) if window and keep else 0
+        gate_stride = gate.stride(0) if gate is not None else 0
+        form = (ctypes.c_float(factor), ctypes.c_float(eps), ctypes.c_float(gain))
+        sizes = (ctypes.c_int(nq), ctypes.c_int(nkv), ctypes.c_int(vd), ctypes.c_int(page_size))
+        mask = (ctypes.c_float(scale), ctypes.c_int(win), ctypes.c_int(keep))
+        n_decode = batch.num_requests - batch.num_prefill_requests
+        paired = (qkv.dtype == torch.bfloat16 and 2 * d == vd and storage is not None
+                  and qkv.shape[1] % 8 == 0)
+        prefill = (paired and self.use_pp_prefill and batch.num_prefill_requests > 0
+                   and bool(self.lib.somi_prefill_pp_supported(*sizes)))
+        decode = (paired and self.use_tma_decode and n_decode > 0
+                  and bool(self.lib.somi_two_map_decode_supported(*sizes)))
+        if prefill or decode:
+            kv_map = ctypes.c_void_p(self._kv_tensor_map(storage, vd, page_size))
+            rows = (ctypes.c_longlong((kcache.data_ptr() - storage.data_ptr()) // (vd * 2)),
+                    ctypes.c_longlong((vcache.data_ptr() - storage.data_ptr()) // (vd * 2)))
+
+        def note(name, first, last, detail=""):
+            if trace.active():
+                moved, flops = self._attention_work(batch, first, last, nq, nkv, vd, qkv.element_size(), win, keep)
+                trace.note(name, moved / (2 * vd) * (2 * d + vd), flops / vd * (d + vd), detail=detail)
+
+        if prefill:
+            tiles = batch.tiles[self.prefill_tc_q_tile]
+            rc = self.lib.somi_two_map_attention_prefill(
+                ctypes.c_void_p(self._q_tensor_map(qkv)), kv_map, *rows, _ptr(group.block_table),
+                ctypes.c_int(group.width), _ptr(batch.cu_q), _ptr(batch.ctx_len), _ptr(tiles),
+                ctypes.c_int(tiles.shape[0]), *sizes, *mask, *form, _ptr(gate),
+                ctypes.c_longlong(gate_stride), _ptr(out), self._stream())
+            self._done(rc, "two_map_attention_prefill")
+            note("two_map_attention_prefill", 0, batch.num_prefill_requests)
+        if decode:
+            # chunks a request reads at most: those of the longest one, or of a window and the kept keys
+            chunk = self.decode_chunk
+            splits = -(-group.width * page_size // chunk)
+            if win:
+                splits = min(splits, (win + chunk - 2) // chunk + 1 + -(-keep // chunk))
+            n_o = n_decode * 2 * nq * splits * vd
+            ws = self._scratch(n_o + n_decode * 2 * nq * splits * 2, qkv.device)
+            rc = self.lib.somi_two_map_attention_decode(
+                kv_map, _ptr(qkv), ctypes.c_int(qkv.shape[1]), ctypes.c_int(batch.num_prefill_tokens),
+                ctypes.c_int(batch.num_prefill_requests), ctypes.c_int(n_decode), *rows,
+                _ptr(group.block_table), ctypes.c_int(group.width), _ptr(batch.ctx_len), *sizes, *mask,
+                *form, _ptr(gate), ctypes.c_longlong(gate_stride), ctypes.c_void_p(ws.data_ptr()),
+                ctypes.c_void_p(ws.data_ptr() + 4 * n_o), ctypes.c_int(splits), _ptr(out), self._stream())
+            self._done(rc, "two_map_attention_decode")
+            self.launches += 1
+            note("two_map_attention_decode", batch.num_prefill_requests, batch.num_requests, "with merge")
+        tiles = batch.tiles[self.generic_q_tile]
+        n_tiles, n_single = 0 if prefill else tiles.shape[0], 0 if decode else n_decode
+        if n_tiles + n_single == 0:
+            return
+        maps = torch.empty((batch.num_tokens, 2 * nq * vd), dtype=torch.float32, device=out.device)
+        rc = self.lib.somi_paged_attention_generic(
+            _ptr(qkv), _code(qkv), ctypes.c_int(qkv.shape[1]), _ptr(kcache), _ptr(vcache),
+            _ptr(group.block_table), ctypes.c_int(group.width), _ptr(batch.cu_q), _ptr(batch.ctx_len),
+            _ptr(tiles), ctypes.c_int(n_tiles), ctypes.c_int(batch.num_prefill_requests),
+            ctypes.c_int(batch.num_prefill_tokens), ctypes.c_int(n_single), ctypes.c_int(2 * nq),
+            ctypes.c_int(nkv), ctypes.c_int(d), ctypes.c_int(vd), ctypes.c_int(page_size),
+            ctypes.c_float(scale), ctypes.c_int(win), ctypes.c_int(0), None, ctypes.c_longlong(0),
+            ctypes.c_int(0), ctypes.c_float(0.0), None, ctypes.c_int(keep), ctypes.c_int(2),
+            ctypes.c_int(1), _ptr(maps), self._stream())
+        self._done(rc, "two_map_attention")
+        note("attention_generic", batch.num_prefill_requests if prefill else 0,
+             batch.num_prefill_requests if decode else batch.num_requests, "two maps")
+        first = batch.num_prefill_tokens if prefill else 0
+        last = batch.num_prefill_tokens if decode else batch.num_tokens
+        rc = self.lib.somi_two_map_difference(
+            _ptr(maps[first:last]), *form, _ptr(gate[first:last] if gate is not None else None),
+            ctypes.c_longlong(gate_stride), ctypes.c_longlong(last - first), ctypes.c_int(nq),
+            ctypes.c_int(vd), _ptr(out[first:last]), _code(out), self._stream())
+        self._done(rc, "two_map_difference")
+        if trace.active():
+            trace.note("two_map_difference", (last - first) * nq * vd * (8 + out.element_size()))
+
+    def head_gate_mul(self, x, gate, heads: int) -> None:
+        """x[t, h * width + i] *= sigmoid(gate[t, h]), in place (`gate`: rows may lie further apart)."""
+        _check(x)
+        if not (gate.is_cuda and gate.dtype == x.dtype and gate.stride(1) == 1
+                and tuple(gate.shape) == (x.shape[0], heads) and x.shape[1] % heads == 0):
+            raise KernelError("a gate per head is [T, heads] of the rows' dtype with contiguous rows")
+        rc = self.lib.somi_head_gate_mul(_ptr(x), _ptr(gate), _code(x), ctypes.c_longlong(gate.stride(0)),
+                                         ctypes.c_longlong(x.shape[0]), ctypes.c_int(heads),
+                                         ctypes.c_int(x.shape[1] // heads), self._stream())
+        self._done(rc, "head_gate_mul")
+        if trace.active():
+            trace.note("head_gate_mul", 2 * x.numel() * x.element_size())
 
     # ------------------------------------------------ gated layers, latent attention
     def embed_sinusoid_layernorm(self, ids, positions, table, inv_freq, weight, eps, out) -> None:
@@ -546,17 +652,18 @@ class CudaOps:
             trace.note("embed_sinusoid_layernorm", ids.shape[0] * table.shape[1] * (table.element_size() + 4))
 
     def add_layernorm(self, residual, delta, gate, weight, eps, out, rows=None, rms=False,
-                      extra=None) -> None:
+                      extra=None, bias=None) -> None:
         """residual += sigmoid(gate) * delta (float32, in place; no gate: plain sum);
-        out = layernorm(residual) * weight (mean taken off; with `rms`, an RMS norm instead).
+        out = layernorm(residual) * weight (+ bias) (mean taken off; with `rms`, an RMS norm instead).
 
         `delta`: [N, H] in the compute dtype, or float32 [splits, N, H] partial sums added in
         order.  `gate`: logits [N, H] whose rows may lie further apart (a view of a wider
         product), or float32 [splits, N, H] partial sums.  `extra`: float32 [N, H] rows that are
         added as well, outside the gate (a second branch of the layer; needs a `delta`).  With
         `rows`, only those rows are produced and residual is not written."""
-        _check(residual, delta, weight, out, rows, extra)
+        _check(residual, delta, weight, out, rows, extra, bias)
         assert residual.dtype == torch.float32
+        assert bias is None or (bias.dtype == weight.dtype and bias.shape == weight.shape)
         assert extra is None or (extra.dtype == torch.float32 and extra.shape == residual.shape
                                  and delta is not None)
         H = residual.shape[1]
@@ -583,7 +690,7 @@ class CudaOps:
             ctypes.c_int(gate_splits), ctypes.c_longlong(gate_split_stride),
             _ptr(weight), _code(weight), ctypes.c_float(eps), _ptr(out), _code(out), _ptr(rows),
             ctypes.c_int(n_out), ctypes.c_int(H), ctypes.c_int(0 if rows is not None else 1),
-            ctypes.c_int(1 if rms else 0), _ptr(extra), self._stream())
+            ctypes.c_int(1 if rms else 0), _ptr(extra), _ptr(bias), self._stream())
         self._done(rc, "add_layernorm")
         if trace.active():
             n = n_out * H
@@ -706,12 +813,14 @@ class CudaOps:
                               "rows up to 1024)")
 
     def latent_rotary_store(self, x, q_at: int, heads: int, q_dim: int, rot: int, c_at: int, rank: int,
-                            positions, inv_freq, neighbours: bool, weight, eps, slot_map, cache, qa) -> None:
+                            positions, inv_freq, neighbours: bool, weight, eps, slot_map, cache, qa,
+                            magnitude: float = 1.0) -> None:
         """Rows of `x` hold, from column `q_at` on, query heads of q_dim + rot elements, and from
         `c_at` on a latent of `rank` elements with a key part of `rot` behind it.  The token's cache
         row [rank + rot] receives rmsnorm(latent) * weight and the turned key part, and
         qa[:, :, rank:] ([heads, T, rank + rot]) every query's turned tail.  Pairs turn by position *
-        inv_freq[i] (float64): neighbours (2i, 2i + 1), or entries i and i + rot / 2."""
+        inv_freq[i] (float64), sine and cosine both times `magnitude`: neighbours (2i, 2i + 1), or
+        entries i and i + rot / 2."""
         _check(positions, inv_freq, weight, slot_map, cache, qa)
         if not (x.is_cuda and x.stride(1) == 1 and x.shape[1] >= max(q_at + heads * (q_dim + rot), c_at + rank + rot)):
             raise KernelError("latent_rotary_store takes a device tensor with contiguous rows")
@@ -724,7 +833,8 @@ class CudaOps:
             _ptr(x), _code(x), ctypes.c_longlong(x.stride(0)), ctypes.c_int(q_at), ctypes.c_int(heads),
             ctypes.c_int(q_dim), ctypes.c_int(rot), ctypes.c_int(c_at), ctypes.c_int(rank),
             ctypes.c_int(1 if neighbours else 0), _ptr(positions), _ptr(inv_freq), _ptr(weight),
-            _code(weight), ctypes.c_float(eps), _ptr(slot_map), _ptr(cache), _ptr(qa), ctypes.c_int(T),
+            _code(weight), ctypes.c_float(eps), ctypes.c_float(magnitude), _ptr(slot_map), _ptr(cache),
+            _ptr(qa), ctypes.c_int(T),
             self._stream())
         self._done(rc, "latent_rotary_store")
         if trace.active():
@@ -995,10 +1105,10 @@ class CudaOps:
 
         `route` = (work, max_tiles) from `moe_route` (None: one group, w [1, N, K], all rows).
         `gather`: row p of the grouped order reads a[entry(p) // top] (else a[p]); `scatter`: it
-        writes out[entry(p)] (else out[p]).  `gated` = (limit, alpha[, shift = 1]): w's rows
-        alternate gate, up and the result is g * sigmoid(alpha * g) * (u + shift) with
-        g = min(gate, limit), u = clamp(up, -limit, limit), N / 2 columns wide (limit infinite,
-        alpha 1, shift 0: silu(gate) * up).  `act` (a name of `ACTIVATIONS`): the result is that
+        writes out[entry(p)] (else out[p]).  `gated` = (limit, alpha[, shift = 1[, cubic = 0]]): w's rows
+        alternate gate, up and the result is g * sigmoid(alpha * (g + cubic * g^3)) * (u + shift)
+        with g = min(gate, limit), u = clamp(up, -limit, limit), N / 2 columns wide (limit
+        infinite, alpha 1, shift 0: silu(gate) * up).  `act` (a name of `ACTIVATIONS`): the result is that
         function of the product, N columns wide (an expert without a gate).  Products are float32
         FMAs summed over K in ascending order."""
         _check(a, w)
@@ -1015,7 +1125,6 @@ class CudaOps:
         assert gated is None or act is None
         out_dtype = torch.float32 if (out_float32 and gated is None and act is None) else a.dtype
         out = torch.empty((n_rows, cols), dtype=out_dtype, device=a.device)
-        limit, alpha, shift = self._gated(gated)
         mode = 1 if gated is not None else (2 if act is not None else 0)
         rc = self.lib.somi_grouped_gemm(
             _ptr(a), _code(a), ctypes.c_longlong(a.stride(0)), ctypes.c_int(top),
@@ -1023,8 +1132,8 @@ class CudaOps:
             ctypes.c_int(n_entries), ctypes.c_int(max_tiles), ctypes.c_int(n_rows), _ptr(out),
             ctypes.c_int(1 if out_dtype == torch.float32 else 0), ctypes.c_longlong(cols),
             ctypes.c_int(1 if scatter else 0), ctypes.c_int(N), ctypes.c_int(K),
-            ctypes.c_int(mode), ctypes.c_float(limit), ctypes.c_float(alpha),
-            ctypes.c_float(shift), ctypes.c_int(self.ACTIVATIONS[act] if act is not None else 0),
+            ctypes.c_int(mode), *self._gated(gated),
+            ctypes.c_int(self.ACTIVATIONS[act] if act is not None else 0),
             self._stream())
         self._done(rc, "grouped_product")
         if trace.active():
@@ -1034,11 +1143,11 @@ class CudaOps:
         return out
 
     @staticmethod
-    def _gated(gated) -> tuple[float, float, float]:
-        """(limit, alpha, shift) of a gated activation; the shift is 1 where it is not given."""
-        if gated is None:
-            return 0.0, 0.0, 0.0
-        return float(gated[0]), float(gated[1]), float(gated[2]) if len(gated) > 2 else 1.0
+    def _gated(gated) -> tuple:
+        """(limit, alpha, shift, cubic) of a gated activation g * sigmoid(alpha * (g + cubic * g^3)) *
+        (u + shift), as the launchers take it; where not given the shift is 1, the cubic term 0."""
+        given = (0.0, 0.0, 0.0) if gated is None else tuple(gated)
+        return tuple(ctypes.c_float(v) for v in (*given, *(1.0, 0.0)[len(given) - 2:]))
 
     @staticmethod
     def _route_parts(route, E: int):
@@ -1061,15 +1170,15 @@ class CudaOps:
             trace.note("moe_gather_rows", 2 * out.numel() * out.element_size())
         return out
 
-    def clamped_gate_up(self, gu, limit: float, alpha: float, shift: float = 1.0) -> torch.Tensor:
-        """Columns of `gu` alternate gate, up: g * sigmoid(alpha * g) * (u + shift) with
-        g = min(gate, limit), u = clamp(up, -limit, limit); float32 arithmetic."""
+    def clamped_gate_up(self, gu, *gated) -> torch.Tensor:
+        """Columns of `gu` alternate gate, up: g * sigmoid(alpha * (g + cubic * g^3)) * (u + shift) with
+        g = min(gate, limit), u = clamp(up, -limit, limit) for `gated` = limit, alpha[, shift = 1[,
+        cubic = 0]]; float32 arithmetic."""
         _check(gu)
         ff = gu.shape[1] // 2
         out = torch.empty((gu.shape[0], ff), dtype=gu.dtype, device=gu.device)
         rc = self.lib.somi_clamped_gate_up(_ptr(gu), _ptr(out), _code(gu), ctypes.c_longlong(gu.shape[0]),
-                                           ctypes.c_int(ff), ctypes.c_float(limit), ctypes.c_float(alpha),
-                                           ctypes.c_float(shift), self._stream())
+                                           ctypes.c_int(ff), *self._gated(gated), self._stream())
         self._done(rc, "clamped_gate_up")
         if trace.active():
             trace.note("clamped_gate_up", 3 * out.numel() * out.element_size())
@@ -1120,7 +1229,7 @@ class CudaOps:
     def moe_gemv(self, a, w, token_ids, table, *, per_token: bool, gated=None, act=None) -> torch.Tensor:
         """A step of few tokens: entry e = (token, k) times the matrix of expert
         table[id[token], k]; w [E, N, K] bfloat16.  `per_token`: a has one row per token (else one
-        per entry).  `gated` = (limit, alpha): rows of w alternate gate, up and the result is the
+        per entry).  `gated` (see `_gated`): rows of w alternate gate, up and the result is the
         experts' activation, bfloat16 [entries, N / 2]; `act` (a name of `ACTIVATIONS`): that
         function of the product, bfloat16 [entries, N]; else float32 [entries, N]."""
         _check(a, w, token_ids, table)
@@ -1137,13 +1246,11 @@ class CudaOps:
             out = torch.empty((n, N), dtype=torch.bfloat16, device=a.device)
         else:
             out = torch.empty((n, N), dtype=torch.float32, device=a.device)
-        limit, alpha, shift = self._gated(gated)
         mode = 1 if gated is not None else (2 if act is not None else 0)
         rc = self.lib.somi_moe_gemv(
             _ptr(a), ctypes.c_longlong(a.stride(0)), ctypes.c_int(top if per_token else 1), _ptr(w),
             _ptr(token_ids), _ptr(table), ctypes.c_int(top), ctypes.c_int(E), ctypes.c_int(n),
-            _ptr(out), ctypes.c_int(N), ctypes.c_int(K), ctypes.c_int(mode),
-            ctypes.c_float(limit), ctypes.c_float(alpha), ctypes.c_float(shift),
+            _ptr(out), ctypes.c_int(N), ctypes.c_int(K), ctypes.c_int(mode), *self._gated(gated),
             ctypes.c_int(self.ACTIVATIONS[act] if act is not None else 0), self._stream())
         self._done(rc, "moe_gemv")
         if trace.active():
@@ -1333,34 +1440,36 @@ class CudaOps:
             trace.note("add_scaled_rmsnorm", moved)
 
     def headnorm_rotary_store(self, qkv, positions, inv_freq, nq, nkv, hd, vd, rotary_dim, q_weight,
-                              k_weight, eps, slot_map, kcache, vcache, magnitude: float = 1.0) -> None:
-        """Rows of `qkv` hold nq query heads and nkv key heads of `hd` elements, then nkv value
-        heads of `vd`.  Every query and key head passes an RMS norm over the head with
+                              k_weight, eps, slot_map, kcache, vcache, magnitude: float = 1.0,
+                              maps: int = 1) -> None:
+        """Rows of `qkv` hold nq query heads and nkv key heads of `hd` elements, then nkv / maps value
+        heads of `vd` (`maps` neighbouring key heads share a cache row [maps * hd] and a value head).  Every query and key head passes an RMS norm over the head with
         `q_weight` / `k_weight` ([hd]; None: no norm); then entry i < rotary_dim / 2 and entry
         i + rotary_dim / 2 turn by position * inv_freq[i] (`inv_freq` float64), sine and cosine
         both multiplied by `magnitude`.  Queries are
         rewritten in place; keys and values go to their cache slots (`slot_map` None: nothing is
         stored)."""
         _check(positions, inv_freq, slot_map, kcache, vcache, q_weight, k_weight)
-        if not (qkv.is_cuda and qkv.stride(1) == 1 and qkv.shape[1] >= (nq + nkv) * hd + nkv * vd):
+        if not (qkv.is_cuda and qkv.stride(1) == 1
+                and qkv.shape[1] >= (nq + nkv) * hd + nkv // maps * vd):
             raise KernelError("headnorm_rotary_store takes a device tensor with contiguous rows")
         assert inv_freq.dtype == torch.float64 and inv_freq.numel() >= max(1, rotary_dim // 2)
         assert (q_weight is None) == (k_weight is None)
         page_size = 1
         if slot_map is not None:
             assert kcache.dtype == qkv.dtype and vcache.dtype == qkv.dtype
-            assert kcache.shape[1] == nkv and kcache.shape[3] == hd and vcache.shape[3] == vd
+            assert kcache.shape[1] == nkv // maps and kcache.shape[3] == maps * hd and vcache.shape[3] == vd
             page_size = kcache.shape[2]
         rc = self.lib.somi_headnorm_rotary_store(
             _ptr(qkv), _code(qkv), ctypes.c_longlong(qkv.stride(0)), _ptr(positions), _ptr(inv_freq),
             ctypes.c_int(qkv.shape[0]), ctypes.c_int(nq), ctypes.c_int(nkv), ctypes.c_int(hd),
             ctypes.c_int(vd), ctypes.c_int(rotary_dim), _ptr(q_weight), _ptr(k_weight),
             ctypes.c_int(_code(q_weight) if q_weight is not None else _F32), ctypes.c_float(eps),
-            ctypes.c_float(magnitude), _ptr(slot_map), _ptr(kcache), _ptr(vcache),
+            ctypes.c_float(magnitude), ctypes.c_int(maps), _ptr(slot_map), _ptr(kcache), _ptr(vcache),
             ctypes.c_int(page_size), self._stream())
         self._done(rc, "headnorm_rotary_store")
         if trace.active():
-            n = qkv.shape[0] * ((nq + nkv) * hd + nkv * vd)
+            n = qkv.shape[0] * ((nq + nkv) * hd + nkv // maps * vd)
             trace.note("headnorm_rotary_store", 2 * n * qkv.element_size())
 
     def check_matrix_state_geometry(self, heads: int, qk_heads: int, dk: int, dv: int) -> None:
@@ -1510,17 +1619,19 @@ class CudaOps:
             trace.note("relu2", 2 * x.numel() * x.element_size())
 
     def moe_router_select(self, logits, correction, count: int, keep: int, top: int,
-                          over_chosen: bool = False, sigmoid: bool = False, group_best: int = 1):
+                          over_chosen: bool = False, sigmoid: bool = False, group_best: int = 1,
+                          outputs: int | None = None, factor: float = 1.0):
         """logits float32 [T, n] -> (chosen int32 [T, top], weight float32 [T, top]): softmax over
         the n outputs; the choice is made on softmax + correction (None: the softmax) among the
         members of the `keep` best of `count` equal groups of neighbours (a group's score is its
         best member's; count <= 1: no groups); the weights are the chosen outputs' softmax.
         `over_chosen`: the `top` largest logits are chosen (no correction, no groups) and the
         weights are the softmax over the chosen logits only.  `sigmoid`: sigmoids of the logits take the
-        softmax's place; `group_best` 2: a group's score is the sum of its two best members'."""
+        softmax's place; `group_best` 2: a group's score is the sum of its two best members'.  `outputs`: only
+        the first so many columns of `logits` are router outputs; `factor` multiplies all weights."""
         _check(logits, correction)
         assert logits.dtype == torch.float32 and (correction is None or correction.dtype == torch.float32)
-        T, n = logits.shape
+        T, n = logits.shape[0], outputs if outputs is not None else logits.shape[1]
         chosen = torch.empty((T, top), dtype=torch.int32, device=logits.device)
         weight = torch.empty((T, top), dtype=torch.float32, device=logits.device)
         rc = self.lib.somi_moe_router_select(_ptr(logits), ctypes.c_longlong(logits.stride(0)),
@@ -1529,28 +1640,44 @@ class CudaOps:
                                              _ptr(chosen), _ptr(weight),
                                              ctypes.c_int(1 if over_chosen else 0),
                                              ctypes.c_int(1 if sigmoid else 0), ctypes.c_int(group_best),
-                                             self._stream())
+                                             ctypes.c_float(factor), self._stream())
         self._done(rc, "moe_router_select")
         if trace.active():
             trace.note("moe_router_select", T * (n * 4 + top * 8))
         return chosen, weight
 
-    def moe_combine_weighted(self, y, place, table, weight, x, num_experts: int) -> torch.Tensor:
+    def moe_combine_weighted(self, y, place, table, weight, x, num_experts: int, side=None,
+                             side_gate=None) -> torch.Tensor:
         """out[t] = sum_k weight[t, k] * (y[row(t * top + k)] if table[t, k] < num_experts else
         x[t]); float32 [T, H].  `place`: the row of every entry where y's rows are in the grouped
-        order (None: row = entry)."""
-        _check(y, place, table, weight, x)
+        order (None: row = entry).  `side`: rows that are added as well, [T, H] or float32
+        [splits, T, H] partial sums, times sigmoid(side_gate[t]) where `side_gate` (float32 [T], a
+        column of a wider product perhaps) is given."""
+        _check(y, place, table, weight, x, side)
         T, top = table.shape
         H = x.shape[1]
         assert y.shape[1] == H and weight.dtype == torch.float32 and table.dtype == torch.int32
+        splits, split_stride = 1, 0
+        if side is not None:
+            assert tuple(side.shape[-2:]) == (T, H)
+            if side.dim() == 3:
+                assert side.dtype == torch.float32
+                splits, split_stride = side.shape[0], T * H
+        if side_gate is not None:
+            assert side_gate.is_cuda and side_gate.dtype == torch.float32 and tuple(side_gate.shape) == (T,)
         out = torch.empty((T, H), dtype=torch.float32, device=x.device)
         rc = self.lib.somi_moe_combine_weighted(_ptr(y), _code(y), _ptr(place), _ptr(table), _ptr(weight),
                                                 _ptr(x), _code(x), ctypes.c_int(num_experts),
                                                 ctypes.c_int(top), ctypes.c_int(T), ctypes.c_int(H),
+                                                _ptr(side), ctypes.c_int(_code(side) if side is not None else _F32),
+                                                ctypes.c_int(splits), ctypes.c_longlong(split_stride),
+                                                _ptr(side_gate),
+                                                ctypes.c_longlong(side_gate.stride(0) if side_gate is not None else 0),
                                                 _ptr(out), self._stream())
         self._done(rc, "moe_combine_weighted")
         if trace.active():
-            trace.note("moe_combine_weighted", T * top * H * y.element_size() + T * H * (4 + x.element_size()))
+            trace.note("moe_combine_weighted", T * top * H * y.element_size() + T * H * (4 + x.element_size())
+                       + (side.numel() * side.element_size() if side is not None else 0))
         return out
 
     def silu_mul(self, gu: torch.Tensor, out: torch.Tensor, interleaved: bool = False) -> None:
@@ -1616,8 +1743,8 @@ class CudaOps:
         mode GEMM_BF16 -> bf16 [M, N] (+ bias); GEMM_F32 -> float32 [M, N];
         GEMM_PARTIAL_F32 -> float32 [splits', M, N] partial sums over ranges of K (bias in the
         first); GEMM_SWIGLU -> bf16 [M, N / 2]: with g the even rows' and u the odd rows' features and
-        `gated` = (limit, alpha, shift), g' * sigmoid(alpha * g') * (u' + shift) where g' = min(g, limit)
-        and u' = u within +-limit (the default is silu(g) * u);
+        `gated` = (limit, alpha, shift[, cubic]), g' * sigmoid(alpha * (g' + cubic g'^3)) * (u' + shift)
+        where g' = min(g, limit) and u' = u within +-limit (the default is silu(g) * u);
         GEMM_XIELU_SIDE -> (bf16 [M, n_act] = xIELU of the first n_act features with the two
         numbers of `act` (float32), bf16 [M, N - n_act] = the other features), bias added to both.
         """
@@ -1651,7 +1778,7 @@ class CudaOps:
                 ctypes.c_int(box), ctypes.c_int(M), ctypes.c_int(N), ctypes.c_int(K),
                 ctypes.c_int(1), ctypes.c_int(mode), _ptr(bias),
                 _code(bias) if bias is not None else _F32, _ptr(out), _ptr(out2),
-                ctypes.c_int(n_act), _ptr(act), *(ctypes.c_float(v) for v in self._gated(gated)),
+                ctypes.c_int(n_act), _ptr(act), *self._gated(gated),
                 ctypes.c_int(1 if deep_ring else 0), self._stream())
         else:
             rc = self.lib.somi_skinny_gemm(
@@ -1659,7 +1786,7 @@ class CudaOps:
                 ctypes.c_int(box), ctypes.c_int(M), ctypes.c_int(N), ctypes.c_int(K),
                 ctypes.c_int(splits), ctypes.c_int(mode), _ptr(bias),
                 _code(bias) if bias is not None else _F32, _ptr(out),
-                *(ctypes.c_float(v) for v in self._gated(gated)),
+                *self._gated(gated),
                 ctypes.c_int(1 if deep_ring else 0), self._stream())
         self._done(rc, "skinny_gemm")
         if trace.active():

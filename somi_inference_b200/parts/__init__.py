@@ -1,7 +1,8 @@
 """Parts of a decoder layer, their registries, and the generic decoder built from them."""
 
-from . import (block, conv_attention, embedding, extras, feedforward, latent, mamba2,  # noqa: F401
-               matrix_state, mixer, moe, norm, normed_attention, position, side_by_side)  # (register kinds)
+from . import (block, conv_attention, differential_attention, embedding, extras,  # noqa: F401
+               feedforward, latent, mamba2, matrix_state, mixer, moe, norm, normed_attention,  # (register kinds)
+               position, side_by_side)
 from .base import (BranchSum, BuildContext, CacheNeeds, GatedDelta, NormedDelta, PagedKVNeeds,
                    ScaledBranches, StateNeeds, TensorDecl)
 from .model import Decoder, declared_tensors

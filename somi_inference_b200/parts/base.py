@@ -91,6 +91,7 @@ class PagedKVNeeds:
     window: int | None = None     # None: all keys; n: only the last n positions are ever read
     value_dim: int | None = None  # width of a value; None: the same as a key's; 0: no values
                                   # are stored (the keys are read as values too)
+    keep_first: int = 0           # beside a window: positions below this stay readable for good
 
     @property
     def value_width(self) -> int:

@@ -15,20 +15,24 @@ from .registry import ARRANGEMENTS
 
 @ARRANGEMENTS.register("pre_norm")
 class PreNormBlock:
+    """A layer without a feed-forward has the mixer's branch only (and one norm)."""
+
     def __init__(self, mixer, feed_forward, norms) -> None:
-        if mixer is None or feed_forward is None:
-            raise ValueError("the pre-norm arrangement needs a mixer and a feed-forward")
-        if set(norms) != {"mixer", "feed_forward"}:
-            raise ValueError("the pre-norm arrangement takes the norms 'mixer' and "
-                             f"'feed_forward', got {sorted(norms)}")
+        if mixer is None:
+            raise ValueError("the pre-norm arrangement needs a mixer")
+        want = {"mixer"} | ({"feed_forward"} if feed_forward is not None else set())
+        if set(norms) != want:
+            raise ValueError(f"the pre-norm arrangement takes the norms {sorted(want)}, got {sorted(norms)}")
         self.mixer = mixer
         self.feed_forward = feed_forward
         self.mixer_norm = norms["mixer"]
-        self.feed_forward_norm = norms["feed_forward"]
+        self.feed_forward_norm = norms.get("feed_forward")
 
     def forward(self, residual, pending, batch, cache, owns_cache):
         h = self.mixer_norm.forward(residual, pending)
         a = self.mixer.forward(h, batch, cache, owns_cache)
+        if self.feed_forward is None:
+            return a
         h = self.feed_forward_norm.forward(residual, a)
         return self.feed_forward.forward(h, batch)
 

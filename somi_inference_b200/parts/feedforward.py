@@ -8,18 +8,39 @@ halves; y = (silu(gate) * up) W_down^T; silu(z) = z * sigmoid(z), in float32.
 
 from __future__ import annotations
 
+import math
+
 import torch
 
 from .base import BuildContext, TensorDecl, names_of
 from .linear import Linear
 from .registry import FEED_FORWARDS
 
+# gated activations by name, as (limit, alpha, shift, cubic) of g sigmoid(alpha (g + cubic g^3)) (u + shift):
+# gelu's tanh form is z sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3))
+GATED_FORMS = {"silu": (math.inf, 1.0, 0.0, 0.0),
+               "gelu_tanh": (math.inf, 2.0 * math.sqrt(2.0 / math.pi), 0.0, 0.044715)}
+
+
+def gated_form(params) -> tuple[float, float, float, float]:
+    """The gated activation that `params` asks for: `activation`, a name of `GATED_FORMS`, or `limit`,
+    `alpha` and `shift`."""
+    name = params.get("activation")
+    if name is not None:
+        if name not in GATED_FORMS:
+            raise ValueError(f"unknown gated activation {name!r} (known: {sorted(GATED_FORMS)})")
+        return GATED_FORMS[name]
+    form = (float(params["limit"]), float(params["alpha"]), float(params["shift"]), 0.0)
+    if not form[0] > 0.0:
+        raise ValueError("the limit of a clamped activation must be positive")
+    return form
 
 
 @FEED_FORWARDS.register("clamped_glu")
 class ClampedGLU:
     """y = W_down (g sigmoid(alpha g) (u + shift)), g = min(W_gate h, limit), u = W_up h within
-    +-limit.  The activation is float32; a step of few tokens makes it in the product's epilogue."""
+    +-limit; or another gated activation by name (see `gated_form`).  The activation is float32; a
+    step of few tokens makes it in the product's epilogue."""
 
     graph_safe = True
 
@@ -34,9 +55,7 @@ class ClampedGLU:
         self.gate_up = Linear(torch.stack([gate, up], dim=1).reshape(2 * gate.shape[0], -1).contiguous(),
                               None, ctx.ops)
         self.down = Linear(tensors[n["down_weight"]], None, ctx.ops)
-        self.gated = (float(params["limit"]), float(params["alpha"]), float(params["shift"]))
-        if not self.gated[0] > 0.0:
-            raise ValueError("the limit of a clamped activation must be positive")
+        self.gated = gated_form(params)
 
     def forward(self, x: torch.Tensor, batch) -> torch.Tensor:
         act = self.gate_up.swiglu(x, self.gated)

@@ -16,11 +16,13 @@ Because k and v are linear in c, the expansions are moved to the query side and 
 so the attention kernel is multi-query attention over the latent cache itself (key = value = c,
 kv_rank wide), and no step ever expands cached positions again.  The two per-head products are
 batched products over heads.  The norms, scores, softmax and sink are float32.
+`gate` = "head": W_g has a row per head, and the logit of a head multiplies all its elements.
 
 Without a query latent (`q_rank` None) queries come straight from the input, q = W_q h, and one product
 makes queries, latent and gate.  With `rot_dim` every query head has rot_dim more elements behind its
 key_dim, W_dkv has rot_dim more rows behind the latent's (they pass no norm), and both turn by
-position (`rotary` = {"dims": rot_dim, "base", "neighbours": pairs (2i, 2i + 1), else halves}):
+position (`rotary` = {"dims": rot_dim, "base", "neighbours": pairs (2i, 2i + 1), else halves; "scaling" as
+`position.rotary_frequencies` takes it, whose magnitude multiplies both turned parts}):
     s = scale * (q_h . k_h + turned(q'_h) . turned(k'))
 with the key part k' shared by the heads.  It is cached behind the latent, so a cache row is
 [c | turned(k')], a query row of the attention kernel [W_uk,h^T q_h | turned(q'_h)], and the values are a row's
@@ -62,7 +64,7 @@ class LatentAttentionMixer:
         if params.get("sink"):
             decl.append(TensorDecl(n["sink"], (H,), init="zeros", matrix=False))
         if params.get("gate"):
-            decl.append(TensorDecl(n["gate"], (H * dv, D)))
+            decl.append(TensorDecl(n["gate"], (H if params["gate"] == "head" else H * dv, D)))
         return decl
 
     def __init__(self, params, tensors, ctx: BuildContext) -> None:
@@ -79,6 +81,9 @@ class LatentAttentionMixer:
         if self.cache_window is not None and (self.window is None or self.window > self.cache_window):
             raise ValueError("a mixer's window cannot reach further back than its cache is kept")
         self.own_latent = bool(params.get("own_latent", True))
+        if params.get("gate") not in (None, False, True, "head"):
+            raise ValueError(f"unknown gate {params['gate']!r} (True: per element, 'head': per head)")
+        self.head_gate = params.get("gate") == "head"
         ctx.ops.check_latent_geometry(H, self.kv_rank, self.rot_dim)
         self.kv_norm = tensors[n["kv_norm"]] if self.own_latent else None
         # W_uk,h^T as rows [kv_rank, key_dim] (q'_h = q_h @ W_uk,h), W_uv,h as rows [value_dim, kv_rank]
@@ -105,9 +110,7 @@ class LatentAttentionMixer:
         rotary = params.get("rotary") or {}
         if int(rotary.get("dims", 0)) != self.rot_dim:
             raise ValueError("the rotation covers exactly the rot_dim part of queries and keys")
-        inv, magnitude = rotary_frequencies(rotary)
-        if magnitude != 1.0:
-            raise ValueError("the rotation of a shared key part takes no magnitude")
+        inv, self.magnitude = rotary_frequencies(rotary)
         self.inv_freq = inv.to(self.ctx.device)
         self.neighbours = bool(rotary.get("neighbours", False))
         weights = [tensors[n["q"]], tensors[n["kv_down"]]]
@@ -137,12 +140,14 @@ class LatentAttentionMixer:
         ops.head_product(q[:, :, :self.key_dim], self.k_up_t, heads_first=True, out=qa[:, :, :R])
         ops.latent_rotary_store(row, 0, H, self.key_dim, rot, self.latent_at, R, batch.positions,
                                 self.inv_freq, self.neighbours, self.kv_norm, self.eps, group.slot_map,
-                                paged.keys, qa)
+                                paged.keys, qa, magnitude=self.magnitude)
         o_lat = torch.empty((H, T, R), dtype=x.dtype, device=x.device)
         ops.latent_attention(qa, paged.keys, batch, group, H, R, self.scale, self.window, self.sinks,
                              o_lat, tail=rot)
         o = ops.head_product(o_lat, self.v_up, heads_first=False).view(T, H * self.value_dim)
-        if self.gate_at is not None:
+        if self.gate_at is not None and self.head_gate:
+            ops.head_gate_mul(o, row[:, self.gate_at:self.gate_at + H], H)
+        elif self.gate_at is not None:
             ops.sigmoid_gate_mul(o, row[:, self.gate_at:self.gate_at + o.shape[1]])
         partial = self.out.partial_sums(o)
         return partial if partial is not None else self.out(o)
@@ -171,7 +176,9 @@ class LatentAttentionMixer:
                              self.sinks, o_lat)
         o = ops.head_product(o_lat, self.v_up, heads_first=False)    # [T, H, value_dim]
         o = o.view(T, H * self.value_dim)
-        if self.gate is not None:
+        if self.gate is not None and self.head_gate:
+            ops.head_gate_mul(o, self.gate(x), H)
+        elif self.gate is not None:
             ops.sigmoid_gate_mul(o, self.gate(x))
         partial = self.out.partial_sums(o)
         return partial if partial is not None else self.out(o)

@@ -59,7 +59,7 @@ class Linear:
                                splits=ops.skinny_splits(x.shape[0], self.out_features, self.in_features))
 
     def swiglu(self, x: torch.Tensor, gated=(float("inf"), 1.0, 0.0)) -> torch.Tensor | None:
-        """silu(gate) * up, or the gated activation (limit, alpha, shift), for a weight whose rows
+        """silu(gate) * up, or the gated activation (limit, alpha, shift[, cubic]), for a weight whose rows
         alternate gate, up; None when not available."""
         if not self.skinny(x):
             return None

@@ -25,6 +25,7 @@ from __future__ import annotations
 import torch
 
 from .base import BuildContext, TensorDecl, names_of
+from .feedforward import gated_form
 from .linear import Linear
 from .registry import FEED_FORWARDS
 
@@ -119,7 +120,11 @@ class RoutedMoE:
     = 2: a group's score is the sum of its two best choices.  `weights` = "softmax_chosen": the `top` largest logits are
     chosen (no correction, no groups) and the weights are the softmax over the chosen logits only.
     `activation` (a name of the kernel table's `ACTIVATIONS`, e.g. "gelu"): experts without a gate,
-    expert(h) = W_down act(W_up h), and no gate tensors.
+    expert(h) = W_down act(W_up h), and no gate tensors.  `gated` = {limit, alpha, shift}: the experts'
+    gated activation is the clamped one of `clamped_glu` instead of silu(gate) * up.  `factor`: all
+    weights are multiplied by it.  `shared` = {"ff", "gated", "token_gate"}: one more gated expert that
+    every token passes, added to the sum; with `token_gate` times sigmoid(W_sg h), one number per token,
+    whose logits are one more column of the router's product.
 
     The router's logits are a float32 product; one kernel makes softmax, choice and weights and
     leaves a table row per token, from which the experts run like those of `table_moe`: entry by
@@ -139,6 +144,13 @@ class RoutedMoE:
             if not params.get("activation"):
                 decl.append(TensorDecl(n["gate"][e], (ff, hidden)))
             decl += [TensorDecl(n["up"][e], (ff, hidden)), TensorDecl(n["down"][e], (hidden, ff))]
+        shared = params.get("shared")
+        if shared:
+            sff = int(shared["ff"])
+            decl += [TensorDecl(n["shared_gate"], (sff, hidden)), TensorDecl(n["shared_up"], (sff, hidden)),
+                     TensorDecl(n["shared_down"], (hidden, sff))]
+            if shared.get("token_gate"):
+                decl.append(TensorDecl(n["shared_token_gate"], (1, hidden)))
         return decl
 
     def __init__(self, params, tensors, ctx: BuildContext) -> None:
@@ -171,31 +183,59 @@ class RoutedMoE:
                              f"{self.group_keep} are kept")
         if self.top > self.group_keep * (self.outputs // self.group_count):
             raise ValueError("the kept groups hold fewer outputs than a token chooses")
-        self.router = Linear(tensors[n["router"]], None, ctx.ops)
+        self.factor = float(params.get("factor", 1.0))
+        router_w = tensors[n["router"]]
+        shared = params.get("shared")
+        self.shared, self.token_gate = None, False
+        if shared:
+            self.shared = (Linear(_interleave(tensors[n["shared_gate"]], tensors[n["shared_up"]]).contiguous(),
+                                  None, ctx.ops),
+                           Linear(tensors[n["shared_down"]], None, ctx.ops), gated_form(shared["gated"]))
+            self.token_gate = bool(shared.get("token_gate"))
+        if self.token_gate:
+            # (rows of zeros behind it keep the logits' rows a multiple of 16 bytes)
+            router_w = torch.cat([router_w, tensors[n["shared_token_gate"]],
+                                  router_w.new_zeros((-(self.outputs + 1) % 8, router_w.shape[1]))], 0).contiguous()
+        self.router = Linear(router_w, None, ctx.ops)
         self.correction = (tensors[n["correction"]].float().contiguous()
                            if params.get("correction") else None)
         E = range(self.experts)
         if self.act is None:
             self.w_gate_up = _interleave(torch.stack([tensors[n["gate"][e]] for e in E]),
                                          torch.stack([tensors[n["up"][e]] for e in E])).contiguous()
-            self.gated = (float("inf"), 1.0, 0.0)           # silu(gate) * up
+            self.gated = gated_form(params.get("gated") or {"activation": "silu"})
         else:
             self.w_gate_up = torch.stack([tensors[n["up"][e]] for e in E]).contiguous()
             self.gated = None
         self.w_down = torch.stack([tensors[n["down"][e]] for e in E]).contiguous()
+
+    def _side(self, x: torch.Tensor, logits: torch.Tensor) -> dict:
+        """The shared expert's result (few tokens: split-K partial sums, added up by the weighted sum)
+        and its gate's logits, as the weighted sum takes them."""
+        if self.shared is None:
+            return {}
+        gate_up, down, form = self.shared
+        act = gate_up.swiglu(x, form)
+        if act is None:
+            act = self.ctx.ops.clamped_gate_up(gate_up(x), *form)
+        side = down.partial_sums(act)
+        return {"side": down(act) if side is None else side,
+                "side_gate": logits[:, self.outputs] if self.token_gate else None}
 
     def forward(self, x: torch.Tensor, batch) -> torch.Tensor:
         ops, top, E = self.ctx.ops, self.top, self.experts
         logits = self.router.to_float32(x)
         chosen, weight = ops.moe_router_select(logits, self.correction, self.group_count,
                                                self.group_keep, top, over_chosen=self.over_chosen,
-                                               sigmoid=self.sigmoid, group_best=self.group_best)
+                                               sigmoid=self.sigmoid, group_best=self.group_best,
+                                               outputs=self.outputs, factor=self.factor)
+        side = self._side(x, logits)
         n_entries = x.shape[0] * top
         if ops.moe_gemv_supported(n_entries, x.shape[1], x.dtype) and self.w_down.shape[2] % 8 == 0:
             act = ops.moe_gemv(x, self.w_gate_up, None, chosen, per_token=True, gated=self.gated,
                                act=self.act)
             y = ops.moe_gemv(act, self.w_down, None, chosen, per_token=False)
-            return ops.moe_combine_weighted(y, None, chosen, weight, x, E)
+            return ops.moe_combine_weighted(y, None, chosen, weight, x, E, **side)
         route = ops.moe_route(None, chosen, E, self.outputs)
         if x.dtype == torch.bfloat16:
             rows = ops.moe_gather_rows(x, route, E, top)
@@ -205,8 +245,9 @@ class RoutedMoE:
                        else ops.unary_act(gu, self.act))
                 y = ops.library_grouped_product(mid, self.w_down, route)
                 if y is not None:
-                    return ops.moe_combine_weighted(y, ops._route_parts(route, E)[2], chosen, weight, x, E)
+                    return ops.moe_combine_weighted(y, ops._route_parts(route, E)[2], chosen, weight, x, E,
+                                                    **side)
         act = ops.grouped_product(x, self.w_gate_up, route=route, top=top, gather=True, gated=self.gated,
                                   act=self.act)
         y = ops.grouped_product(act, self.w_down, route=route, top=top, scatter=True, out_float32=True)
-        return ops.moe_combine_weighted(y, None, chosen, weight, x, E)
+        return ops.moe_combine_weighted(y, None, chosen, weight, x, E, **side)

@@ -124,21 +124,26 @@ class NoNorm:
 
 @NORMS.register("layernorm")
 class LayerNorm:
-    """(x - mean) / sqrt(var + eps) * weight, var the mean of the squared deviations; a weight and
-    no bias.  Mean, variance and the residual sum are float32.  `delta` may be a `GatedDelta`:
+    """(x - mean) / sqrt(var + eps) * weight, var the mean of the squared deviations; plus a bias
+    where `names` has one.  Mean, variance and the residual sum are float32.  `delta` may be a `GatedDelta`:
     the branch's result is then multiplied by sigmoid(gate logits) as it is added; or a
     `BranchSum`: both results of the layer before are added."""
 
     @staticmethod
     def declare(params) -> list[TensorDecl]:
-        return [TensorDecl(names_of(params)["weight"], (int(params["size"]),), init="ones",
-                           matrix=False)]
+        n, shape = names_of(params), (int(params["size"]),)
+        decl = [TensorDecl(n["weight"], shape, init="ones", matrix=False)]
+        if "bias" in n:
+            decl.append(TensorDecl(n["bias"], shape, init="zeros", matrix=False))
+        return decl
 
     def __init__(self, params, tensors, ctx: BuildContext) -> None:
+        n = names_of(params)
         self.size = int(params["size"])
         self.eps = float(params["eps"])
         self.ctx = ctx
-        self.weight = tensors[names_of(params)["weight"]]
+        self.weight = tensors[n["weight"]]
+        self.bias = tensors[n["bias"]].to(self.weight.dtype) if "bias" in n else None
 
     def forward(self, residual: torch.Tensor, delta=None,
                 rows: torch.Tensor | None = None) -> torch.Tensor:
@@ -152,5 +157,5 @@ class LayerNorm:
         n = residual.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((n, self.size), dtype=self.ctx.dtype, device=residual.device)
         self.ctx.ops.add_layernorm(residual, delta, gate, self.weight, self.eps, out, rows,
-                                   extra=extra)
+                                   extra=extra, bias=self.bias)
         return out
