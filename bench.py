@@ -9,6 +9,7 @@
     python bench.py --arch poselorn --only decode|prefill [...]  the same shapes with Poselorn layers
     python bench.py --arch gikarax --only decode|prefill [...]   the same shapes with Gikarax layers
     python bench.py --arch dosuvik --only decode|prefill [...]   the same shapes with Dosuvik layers
+    python bench.py --arch bibalix --only decode|prefill [...]   the same shapes with Bibalix layers
 
 A step is one decode step of the whole engine: 8 requests with 2,048 cached tokens each,
 random bfloat16 weights, one new token per request (batch layout upload, all layers, head,
@@ -91,6 +92,13 @@ GIKARAX = dict(window=8192, softcap=30.0, rank=128, tau=8.0, experts=16, top=4)
 # heads at the same widths; sixteen experts of a quarter of the dense feed-forward's width in four
 # groups of which two are kept, four per token.
 DOSUVIK = dict(window=8192, limit=7.0, experts=16, top=4, groups=(4, 2))
+# `--arch bibalix`: the same widths, head counts and vocabularies with Bibalix layers in the pattern
+# attention in two maps + dense, latent attention + experts (twice), attention in two maps + experts:
+# values of the shape's head size under two keys of half of it (a cache row is as long as the Qwen2
+# layer's), windows longer than the timed contexts beside 64 kept tokens; Digosun's key/value latents with
+# a rotated key part of half a head; sixteen experts of a quarter of the dense feed-forward's width,
+# four per token, beside a shared expert of the same width.
+BIBALIX = dict(window=8192, keep=64, diff=0.5, limit=7.0, experts=16, top=4, factor=2.0)
 CONTEXT = 2048          # cached tokens per request when decode is timed
 MAX_CONTEXT = 4096      # "benchmark at context 4096": positions the model is laid out for
 LONG_CONTEXT = 40960    # ... when the points at 8 k and 32 k cached tokens are measured too
@@ -331,13 +339,34 @@ def dosuvik_config(shape: str, layers: int, positions: int) -> dict:
             "layers": [dict(zip(("type", "mixer", "mlp"), pattern[i % 4])) for i in range(layers)]}
 
 
+def bibalix_config(shape: str, layers: int, positions: int) -> dict:
+    q, z = SHAPES[shape], BIBALIX
+    D, hd, H, G = q["hidden_size"], q["head_dim"], q["num_attention_heads"], q["num_key_value_heads"]
+    maps = dict(heads=H, kv_heads=G, dim=hd // 2, vdim=hd, scale=(hd // 2) ** -0.5, diff=z["diff"],
+                mask={"size": z["window"], "keep_first": z["keep"]},
+                rot={"dims": hd // 2, "base": q["rope_theta"]})
+    latent = dict(heads=H, dim=hd, rot_dim=hd // 2, vdim=hd, kv_rank=DIGOSUN_SHAPES[shape]["kv_rank"],
+                  scale=(1.5 * hd) ** -0.5, mask={"size": z["window"]},
+                  rot={"dims": hd // 2, "base": q["rope_theta"],
+                       "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}})
+    dense = {"kind": "dense", "ff": q["intermediate_size"]}
+    expert = {"ff": q["intermediate_size"] // 4, "limit": z["limit"]}
+    moe = {"kind": "moe", "expert": expert, "shared": expert,
+           "router": {"experts": z["experts"], "top": z["top"], "scale": z["factor"]}}
+    pattern = [("attention", maps, dense), ("latent_attention", latent, moe),
+               ("latent_attention", latent, moe), ("attention", maps, moe)]
+    return {"architecture": "Bibalix", "vocab": q["vocab_size"], "width": D,
+            "norm": {"eps": q["rms_norm_eps"]}, "max_positions": positions,
+            "layers": [dict(zip(("type", "mixer", "mlp"), pattern[i % 4])) for i in range(layers)]}
+
+
 ARCH = "qwen2"     # set by --arch; the other architectures build the same shapes with their layers
 
 
 def build_engine(shape: str, layers: int, max_tokens: int, max_requests: int, positions: int):
     import torch
 
-    from somi_inference_b200.config import (DapozenConfig, DigosunConfig, DosuvikConfig,
+    from somi_inference_b200.config import (BibalixConfig, DapozenConfig, DigosunConfig, DosuvikConfig,
                                             GikaraxConfig, PoselornConfig, Qwen2Config)
     from somi_inference_b200.engine import Engine
     from somi_inference_b200.parts import declared_tensors
@@ -351,6 +380,8 @@ def build_engine(shape: str, layers: int, max_tokens: int, max_requests: int, po
         cfg = GikaraxConfig.from_dict(gikarax_config(shape, layers, positions))
     elif ARCH == "dosuvik":
         cfg = DosuvikConfig.from_dict(dosuvik_config(shape, layers, positions))
+    elif ARCH == "bibalix":
+        cfg = BibalixConfig.from_dict(bibalix_config(shape, layers, positions))
     else:
         cfg = Qwen2Config.from_dict(shape_config(shape, layers, positions))
     gen = torch.Generator(device="cuda").manual_seed(0)
@@ -597,7 +628,53 @@ def dosuvik_sizes(cfg, batch: int) -> dict:
             "state_bytes_per_request": state, "window": min(windows)}
 
 
+def bibalix_sizes(cfg, batch: int) -> dict:
+    """The same figures for a Bibalix model.  A decode step of `batch` tokens reads at most
+    batch * top routed experts of a layer and its shared expert; a latent cache row holds kv_rank + rot_dim
+    numbers, read once for all heads; a two-map cache row two keys and one value per key/value head,
+    and a (query, key) pair of a head takes two scores and two weighted values."""
+    D, V = cfg.width, cfg.vocab
+    params = read_params = small = kv = pair = 0
+    windows = [1 << 30]
+    for layer in cfg.layers:
+        m = layer.mixer
+        if layer.type == "latent_attention":
+            p = (m["heads"] * (m["dim"] + m["rot_dim"] + m["vdim"] + 1) + m["kv_rank"] + m["rot_dim"]) * D \
+                + m["heads"] * (m["dim"] + m["vdim"]) * m["kv_rank"]
+            small += m["kv_rank"]
+            kv += 2 * (m["kv_rank"] + m["rot_dim"])
+            pair += 2 * m["heads"] * (2 * m["kv_rank"] + m["rot_dim"])
+        else:
+            qk, v = 2 * (m["heads"] + m["kv_heads"]) * m["dim"], m["kv_heads"] * m["vdim"]
+            p = (qk + v + m["heads"] * (m["vdim"] + 1)) * D
+            small += qk + v + 2 * m["dim"]
+            kv += 2 * m["kv_heads"] * (2 * m["dim"] + m["vdim"])
+            pair += 4 * m["heads"] * (m["dim"] + m["vdim"])
+        if m.get("mask"):
+            windows.append(m["mask"]["size"])
+        params += p
+        read_params += p
+        small += 4 * D
+        mlp = layer.mlp
+        if mlp is None:
+            continue
+        if mlp["kind"] == "dense":
+            params += 3 * D * mlp["ff"]
+            read_params += 3 * D * mlp["ff"]
+        else:
+            r = mlp["router"]
+            one = 3 * D * mlp["expert"]["ff"]
+            every = r["experts"] * D + (3 * D * mlp["shared"]["ff"] + D if mlp.get("shared") else 0)
+            params += r["top"] * one + every
+            read_params += min(r["experts"], batch * r["top"]) * one + every
+    return {"weight_bytes": 2 * (read_params + small + V * D + 2 * D), "kv_bytes_per_token": kv,
+            "matmul_params": params, "head_params": V * D, "attn_flops_per_pair": pair,
+            "window": min(windows)}
+
+
 def model_sizes(cfg, layers: int, batch: int = 1) -> dict:
+    if ARCH == "bibalix":
+        return bibalix_sizes(cfg, batch)
     if ARCH == "dosuvik":
         return dosuvik_sizes(cfg, batch)
     if ARCH == "gikarax":
@@ -1199,7 +1276,7 @@ def main() -> int:
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", choices=["ours", "reference"], default="ours")
     ap.add_argument("--shape", choices=list(SHAPES), default="7b")
-    ap.add_argument("--arch", choices=["qwen2", "digosun", "dapozen", "poselorn", "gikarax", "dosuvik"],
+    ap.add_argument("--arch", choices=["qwen2", "digosun", "dapozen", "poselorn", "gikarax", "dosuvik", "bibalix"],
                     default="qwen2",
                     help="with --only decode|prefill: the layer design the shape is built with "
                          "(digosun: latent attention under a window, gated branches; dapozen: "
@@ -1207,7 +1284,8 @@ def main() -> int:
                          "gikarax: latent, capped window and causal attention, a gated linear "
                          "attention, experts without gates, a loop; dosuvik: window attention with "
                          "turned values, retention, latent attention with a rotated key part, norms "
-                         "behind the branches, averages over depth)")
+                         "behind the branches, averages over depth; bibalix: attention in two maps "
+                         "beside kept first tokens, latent attention under a window, a shared expert)")
     ap.add_argument("--layers", type=int, default=None, help="fewer layers than the shape has")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--no-points", action="store_true",

@@ -54,12 +54,12 @@ struct TdRange {
         return p0 < kv_len && (p0 + page_size > first_key || p0 < keep);
     }
 };
-__device__ __forceinline__ TdRange td_range(int ctx_len, int window, int keep) {
+__device__ __forceinline__ TdRange td_range(int ctx_len, int window, int keep, bool compact) {
     TdRange r;
     r.kv_len = ctx_len + 1;
     r.first_key = first_visible_key(ctx_len, window);
     r.keep = keep;
-    const KeptSplits k = kept_splits(r.first_key, r.kv_len, keep, kTdChunk);
+    const KeptSplits k = kept_splits(r.first_key, r.kv_len, keep, kTdChunk, compact);
     r.first_split = k.first;
     r.n_splits = k.end;
     r.n_keep = k.n_keep;
@@ -100,7 +100,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map,
     const int split = blockIdx.x, kvh = blockIdx.y, i = blockIdx.z;
     const int req = req_base + i, row = row_base + i;
     const int G = nq / nkv * maps;                                    // MMA rows in use
-    const TdRange rg = td_range(ld_step(ctx_len + req), window, keep);      // before the wait
+    const TdRange rg = td_range(ld_step(ctx_len + req), window, keep, maps > 1);      // before the wait
     if (split < rg.first_split || split >= rg.n_splits) {
         pdl_wait();
         return;
@@ -349,7 +349,7 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
     const int group = blockIdx.x, kvh = blockIdx.y, i = blockIdx.z;
     const int req = req_base + i, row = row_base + i;
     const int G = nq / nkv * maps;                                    // MMA rows in use
-    const TdRange rg = td_range(ld_step(ctx_len + req), window, keep);      // before the wait
+    const TdRange rg = td_range(ld_step(ctx_len + req), window, keep, maps > 1);      // before the wait
     const int c_begin = max(group * cpc, rg.first_split);
     const int c_end = min((group + 1) * cpc, rg.n_splits);
     if (c_begin >= c_end) {

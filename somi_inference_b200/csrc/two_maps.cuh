@@ -18,14 +18,16 @@ struct TwoMaps {
 };
 
 // Chunks of `chunk` keys that hold [0, keep) or [first_key, kv_len), numbered first .. end - 1: number
-// s is chunk s below n_keep and chunk s + gap from there on.
+// s is chunk s below n_keep and chunk s + gap from there on.  `compact`: numbered from 0 on without
+// those between the kept keys and the window; else (no kept keys) by their place in the sequence.
 struct KeptSplits {
     int first, end, n_keep, gap;
 };
-__device__ __forceinline__ KeptSplits kept_splits(int first_key, int kv_len, int keep, int chunk) {
+__device__ __forceinline__ KeptSplits kept_splits(int first_key, int kv_len, int keep, int chunk,
+                                                  bool compact) {
     KeptSplits k;
     const int first = first_key / chunk, last = (kv_len + chunk - 1) / chunk;
-    if (keep <= 0) {
+    if (!compact) {
         k.first = first;
         k.end = last;
         k.n_keep = k.gap = 0;
@@ -66,7 +68,7 @@ two_map_merge_kernel(const float* __restrict__ part_o, const float* __restrict__
     const int i = blockIdx.x, head = blockIdx.y;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, map = warp & 1;
     const int ctx = ctx_len[req_base + i];
-    const KeptSplits k = kept_splits(first_visible_key(ctx, window), ctx + 1, keep, chunk);
+    const KeptSplits k = kept_splits(first_visible_key(ctx, window), ctx + 1, keep, chunk, true);
     const int first = k.first / cpc, end = (k.end + cpc - 1) / cpc;
     const size_t base = (static_cast<size_t>(i) * 2 * nq + 2 * head + map) * max_splits;
     float M = -INFINITY;
