@@ -12,7 +12,7 @@
 //
 // Needs head_dim 64 or 128 and a page size that is a multiple of 8 and divides 128.
 //
-// `maps` = 2: a key row of head_dim elements holds two keys of half that width over one value
+// TWO_MAPS: a key row of head_dim elements holds two keys of half that width over one value
 // (attention in two maps, see two_maps.cuh).  Every head of the group is then two MMA rows, its
 // query's first half with zeros behind it and its second half with zeros in front, so the
 // scores of both maps come from one product over the same key tile; the merge takes the
@@ -41,25 +41,30 @@ __device__ __forceinline__ int tma_tile_offset(int key, int chunk) {
 }
 
 // The keys of a request: [0, keep) and [first_key, kv_len), and its chunks, numbered from
-// first_split to n_splits with those between the kept ones and the window's left out.
+// first_split to n_splits with those between the kept ones and the window's left out.  KEPT false: no
+// key is kept beside the window, and the chunks are numbered by their place.
+template <bool KEPT>
 struct TdRange {
     int kv_len, first_key, keep, first_split, n_splits, n_keep, gap;
-    __device__ __forceinline__ int chunk_of(int split) const { return split < n_keep ? split : split + gap; }
+    __device__ __forceinline__ int chunk_of(int split) const {
+        return !KEPT || split < n_keep ? split : split + gap;
+    }
     __device__ __forceinline__ bool sees(int key) const {
-        return key < kv_len && (key >= first_key || key < keep);
+        return key < kv_len && (key >= first_key || (KEPT && key < keep));
     }
     // whether a page holds keys that are read
     __device__ __forceinline__ bool needs(int page, int page_size) const {
         const int p0 = page * page_size;
-        return p0 < kv_len && (p0 + page_size > first_key || p0 < keep);
+        return p0 < kv_len && (p0 + page_size > first_key || (KEPT && p0 < keep));
     }
 };
-__device__ __forceinline__ TdRange td_range(int ctx_len, int window, int keep, bool compact) {
-    TdRange r;
+template <bool KEPT>
+__device__ __forceinline__ TdRange<KEPT> td_range(int ctx_len, int window, int keep) {
+    TdRange<KEPT> r;
     r.kv_len = ctx_len + 1;
     r.first_key = first_visible_key(ctx_len, window);
     r.keep = keep;
-    const KeptSplits k = kept_splits(r.first_key, r.kv_len, keep, kTdChunk, compact);
+    const KeptSplits k = kept_splits(r.first_key, r.kv_len, keep, kTdChunk, KEPT);
     r.first_split = k.first;
     r.n_splits = k.end;
     r.n_keep = k.n_keep;
@@ -67,14 +72,14 @@ __device__ __forceinline__ TdRange td_range(int ctx_len, int window, int keep, b
     return r;
 }
 
-template <int HD>
+template <int HD, bool TWO_MAPS>
 __global__ void __launch_bounds__(kTdThreads, 3)
 paged_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map,
                         const __nv_bfloat16* __restrict__ qkv, int row_stride, int row_base,
                         int req_base, long long k_row0, long long v_row0,
                         const int* __restrict__ block_table, int bt_stride,
                         const int* __restrict__ ctx_len, int nq, int nkv, int page_size,
-                        float scale_log2e, int window, int keep, int maps, float* __restrict__ part_o,
+                        float scale_log2e, int window, int keep, float* __restrict__ part_o,
                         float* __restrict__ part_ml, int max_splits, int merge_all,
                         __nv_bfloat16* __restrict__ out) {
     constexpr int CPR = HD / 8;
@@ -99,8 +104,9 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap kv_map,
 
     const int split = blockIdx.x, kvh = blockIdx.y, i = blockIdx.z;
     const int req = req_base + i, row = row_base + i;
+    constexpr int maps = TWO_MAPS ? 2 : 1;
     const int G = nq / nkv * maps;                                    // MMA rows in use
-    const TdRange rg = td_range(ld_step(ctx_len + req), window, keep, maps > 1);      // before the wait
+    const TdRange<TWO_MAPS> rg = td_range<TWO_MAPS>(ld_step(ctx_len + req), window, keep);      // before the wait
     if (split < rg.first_split || split >= rg.n_splits) {
         pdl_wait();
         return;
@@ -321,14 +327,14 @@ __device__ __forceinline__ void ring_compute_sync() {         // the four comput
 constexpr int kRingMaxCpc = 8;
 static int g_ring_chunks = 0;           // chunks per CTA; 0: chosen from the step's size
 
-template <int HD>
+template <int HD, bool TWO_MAPS>
 __global__ void __launch_bounds__(kRingThreads)
 paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
                          const __nv_bfloat16* __restrict__ qkv, int row_stride, int row_base,
                          int req_base, long long k_row0, long long v_row0,
                          const int* __restrict__ block_table, int bt_stride,
                          const int* __restrict__ ctx_len, int nq, int nkv, int page_size,
-                         float scale_log2e, int window, int keep, int maps, float* __restrict__ part_o,
+                         float scale_log2e, int window, int keep, float* __restrict__ part_o,
                          float* __restrict__ part_ml, int max_splits, int cpc, int merge_all,
                          __nv_bfloat16* __restrict__ out) {
     constexpr int CPR = HD / 8;
@@ -348,8 +354,9 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
 
     const int group = blockIdx.x, kvh = blockIdx.y, i = blockIdx.z;
     const int req = req_base + i, row = row_base + i;
+    constexpr int maps = TWO_MAPS ? 2 : 1;
     const int G = nq / nkv * maps;                                    // MMA rows in use
-    const TdRange rg = td_range(ld_step(ctx_len + req), window, keep, maps > 1);      // before the wait
+    const TdRange<TWO_MAPS> rg = td_range<TWO_MAPS>(ld_step(ctx_len + req), window, keep);      // before the wait
     const int c_begin = max(group * cpc, rg.first_split);
     const int c_end = min((group + 1) * cpc, rg.n_splits);
     if (c_begin >= c_end) {
@@ -588,7 +595,7 @@ paged_decode_ring_kernel(const __grid_constant__ CUtensorMap kv_map,
         }
     }
 }
-template <int HD>
+template <int HD, bool TWO_MAPS = false>
 int launch_tma_decode(const CUtensorMap* map, const void* qkv, int row_stride, int row_base,
                       int req_base, int n_decode, long long k_row0, long long v_row0,
                       const int* block_table, int bt_stride, const int* ctx_len, int nq, int nkv,
@@ -597,12 +604,11 @@ int launch_tma_decode(const CUtensorMap* map, const void* qkv, int row_stride, i
                       const float* turn, int keep = 0, const TwoMaps* two = nullptr) {
     // sinks, turned outputs and differences of maps are the merge kernel's: every request goes
     // through it then
-    const int merge_all = sinks != nullptr || turn != nullptr || two != nullptr;
-    const int maps = two != nullptr ? 2 : 1;
+    const int merge_all = TWO_MAPS || sinks != nullptr || turn != nullptr;
     constexpr int TILE = (HD / 64) * kHalfBytes;
     const size_t smem = 2 * TILE + kTdRows * HD * 2 + kTdRows * kTdChunk * 2 + 1024;
-    cudaFuncSetAttribute(paged_decode_tma_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                         (int)smem);
+    cudaFuncSetAttribute(paged_decode_tma_kernel<HD, TWO_MAPS>,
+                         cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     // Many chunks per SM: CTAs that walk through several chunks each (see the ring kernel).
     static int sm_count = 0;
     if (sm_count == 0) {
@@ -618,16 +624,16 @@ int launch_tma_decode(const CUtensorMap* map, const void* qkv, int row_stride, i
                         : static_cast<int>(std::min<long long>(kRingMaxCpc, units / (8LL * sm_count)));
     if (cpc >= 2) {
         const size_t ring_smem = (kRingK + kRingV) * TILE + kTdRows * HD * 2 + kTdRows * kTdChunk * 2 + 1024;
-        cudaFuncSetAttribute(paged_decode_ring_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                             (int)ring_smem);
+        cudaFuncSetAttribute(paged_decode_ring_kernel<HD, TWO_MAPS>,
+                             cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ring_smem);
         const int groups = (max_splits + cpc - 1) / cpc;
-        launch_pdl(paged_decode_ring_kernel<HD>, dim3(groups, nkv, n_decode), dim3(kRingThreads),
+        launch_pdl(paged_decode_ring_kernel<HD, TWO_MAPS>, dim3(groups, nkv, n_decode), dim3(kRingThreads),
                    ring_smem, stream, *map, static_cast<const __nv_bfloat16*>(qkv), row_stride,
                    row_base, req_base, k_row0, v_row0, block_table, bt_stride, ctx_len, nq, nkv,
-                   page_size, scale * 1.4426950408889634f, window, keep, maps, part_o, part_ml, max_splits,
+                   page_size, scale * 1.4426950408889634f, window, keep, part_o, part_ml, max_splits,
                    cpc, merge_all, static_cast<__nv_bfloat16*>(out));
         int rc = launch_status();
-        if (rc == 0 && two != nullptr)
+        if (TWO_MAPS && rc == 0)
             return launch_two_map_merge<HD>(part_o, part_ml, max_splits, kTdChunk, cpc, ctx_len, row_base,
                                             req_base, n_decode, nq, window, keep, *two,
                                             static_cast<__nv_bfloat16*>(out), stream);
@@ -637,13 +643,13 @@ int launch_tma_decode(const CUtensorMap* map, const void* qkv, int row_stride, i
                                        static_cast<__nv_bfloat16*>(out), stream, sinks, turn, merge_all);
     }
     dim3 grid(max_splits, nkv, n_decode);
-    launch_pdl(paged_decode_tma_kernel<HD>, dim3(grid), dim3(kTdThreads), smem, stream, 
+    launch_pdl(paged_decode_tma_kernel<HD, TWO_MAPS>, dim3(grid), dim3(kTdThreads), smem, stream, 
         *map, static_cast<const __nv_bfloat16*>(qkv), row_stride, row_base, req_base, k_row0,
         v_row0, block_table, bt_stride, ctx_len, nq, nkv, page_size,
-        scale * 1.4426950408889634f, window, keep, maps, part_o, part_ml, max_splits, merge_all,
+        scale * 1.4426950408889634f, window, keep, part_o, part_ml, max_splits, merge_all,
         static_cast<__nv_bfloat16*>(out));
     int rc = launch_status();
-    if (rc == 0 && two != nullptr)
+    if (TWO_MAPS && rc == 0)
         return launch_two_map_merge<HD>(part_o, part_ml, max_splits, kTdChunk, 1, ctx_len, row_base, req_base,
                                         n_decode, nq, window, keep, *two, static_cast<__nv_bfloat16*>(out),
                                         stream);
@@ -726,11 +732,11 @@ SOMI_API int somi_two_map_attention_decode(
     const CUtensorMap* map = static_cast<const CUtensorMap*>(tensor_map);
     const TwoMaps two{factor, eps, gain, gate, gate_stride};
     if (hd == 64)
-        return launch_tma_decode<64>(map, qkv, row_stride, row_base, req_base, n_decode, k_row0,
+        return launch_tma_decode<64, true>(map, qkv, row_stride, row_base, req_base, n_decode, k_row0,
                                      v_row0, block_table, bt_stride, ctx_len, nq, nkv, page_size, scale,
                                      window, part_o, part_ml, max_splits, out, stream, nullptr, nullptr,
                                      keep, &two);
-    return launch_tma_decode<128>(map, qkv, row_stride, row_base, req_base, n_decode, k_row0, v_row0,
+    return launch_tma_decode<128, true>(map, qkv, row_stride, row_base, req_base, n_decode, k_row0, v_row0,
                                   block_table, bt_stride, ctx_len, nq, nkv, page_size, scale, window,
                                   part_o, part_ml, max_splits, out, stream, nullptr, nullptr, keep, &two);
 }

@@ -388,25 +388,41 @@ __global__ void moe_combine_kernel(const TY* __restrict__ y, const int* __restri
 // themselves (no correction, no groups) and the weights are the softmax over the chosen logits only.
 // `sigmoid`: s = sigmoid(logits) instead of the softmax; `group_best` 2: a group's score is the sum of
 // its two largest choices (of its only one where it has one member).  All weights are multiplied by `factor`.
+// The logits may be `splits` partial sums `split_stride` apart, added in order.  `tail` (or null): receives
+// the column behind the outputs, summed likewise (the logit of a gate that rides on the product).
 __global__ void moe_router_select_kernel(const float* __restrict__ logits, long long l_stride,
+                                         int splits, long long split_stride,
                                          const float* __restrict__ correction, int n, int count,
                                          int keep, int top, int* __restrict__ chosen,
                                          float* __restrict__ weight, int T, int over_chosen,
-                                         int sigmoid, int group_best, float factor) {
-    extern __shared__ float rs[];            // per warp: s [n], choice [n], group score [count]
+                                         int sigmoid, int group_best, float factor,
+                                         float* __restrict__ tail) {
+    extern __shared__ float rs[];            // per warp: s [n], choice [n], logits [n], group score [count]
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int t = blockIdx.x * (blockDim.x >> 5) + warp;
     if (t >= T) return;
     const int groups = count > 1 ? count : 1;
-    float* sv = rs + static_cast<size_t>(warp) * (2 * n + groups);
+    float* sv = rs + static_cast<size_t>(warp) * (3 * n + groups);
     float* cv = sv + n;
-    float* gv = cv + n;
-    const float* z = logits + static_cast<size_t>(t) * l_stride;
+    float* z = cv + n;
+    float* gv = z + n;
+    const float* row = logits + static_cast<size_t>(t) * l_stride;
     float m = -INFINITY;
-    for (int i = lane; i < n; i += 32) m = fmaxf(m, z[i]);
+    for (int i = lane; i < n + (tail != nullptr ? 1 : 0); i += 32) {
+        float v = row[i];
+#pragma unroll 8
+        for (int sp = 1; sp < splits; ++sp) v += row[sp * split_stride + i];
+        if (i == n) {
+            tail[t] = v;
+        } else {
+            z[i] = v;
+            m = fmaxf(m, v);
+        }
+    }
     m = warp_max(m);
+    __syncwarp();
     float sum = 0.f;
     for (int i = lane; i < n; i += 32) {
         const float e = sigmoid ? 1.0f / (1.0f + expf(-z[i])) : expf(z[i] - m);
@@ -488,8 +504,9 @@ __global__ void moe_router_select_kernel(const float* __restrict__ logits, long 
 // `side` (or null): the result of an expert that every token passes, [side_splits] partial sums (TS) that
 // lie `side_stride` elements apart and are added in order; with `side_gate` (float32, tokens
 // `gate_stride` apart) it joins the sum times sigmoid(side_gate[t]).
-// A CTA per token (its entries of table, weight and place are read once by every warp); a thread
-// four neighbouring columns where the rows allow it (`vec`), else one.
+// A CTA per token (its entries of table, weight and place are read once by every warp), or several
+// that share its columns (grid.y) in steps of few tokens; a thread four neighbouring columns where
+// the rows allow it (`vec`), else one.
 template <typename TY, typename TX, typename TS>
 __global__ void moe_combine_weighted_kernel(const TY* __restrict__ y, const int* __restrict__ place,
                                             const int* __restrict__ table,
@@ -506,7 +523,7 @@ __global__ void moe_combine_weighted_kernel(const TY* __restrict__ y, const int*
         float* o = out + static_cast<size_t>(t) * H;
         const float sg = side_gate != nullptr ? 1.0f / (1.0f + expf(-side_gate[t * gate_stride])) : 1.0f;
         if (vec) {
-            for (int c = 4 * threadIdx.x; c < H; c += 4 * blockDim.x) {
+            for (int c = 4 * (blockIdx.y * blockDim.x + threadIdx.x); c < H; c += 4 * blockDim.x * gridDim.y) {
                 F4 s{{0.f, 0.f, 0.f, 0.f}};
                 for (int k = 0; k < top; ++k) {
                     const int expert = table[e0 + k];
@@ -519,6 +536,7 @@ __global__ void moe_combine_weighted_kernel(const TY* __restrict__ y, const int*
                 }
                 if (side != nullptr) {
                     F4 d = load4(side + static_cast<size_t>(t) * H + c);
+#pragma unroll 4
                     for (int sp = 1; sp < side_splits; ++sp) {
                         const F4 v = load4(side + sp * side_stride + static_cast<size_t>(t) * H + c);
 #pragma unroll
@@ -530,7 +548,7 @@ __global__ void moe_combine_weighted_kernel(const TY* __restrict__ y, const int*
                 store4(o + c, s);
             }
         } else {
-            for (int c = threadIdx.x; c < H; c += blockDim.x) {
+            for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < H; c += blockDim.x * gridDim.y) {
                 float s = 0.f;
                 for (int k = 0; k < top; ++k) {
                     const int expert = table[e0 + k];
@@ -717,23 +735,24 @@ SOMI_API int somi_moe_combine(const void* y, int y_dtype, const int* place, cons
     return launch_status();
 }
 
-// logits: float32 [T, l_stride] (n columns read); chosen int32 [T, top], weight float32 [T, top].
-SOMI_API int somi_moe_router_select(const float* logits, long long l_stride, const float* correction,
+// logits: float32 [splits, T, l_stride] (n columns read, and one more with `tail`); chosen int32 [T, top], weight float32 [T, top].
+SOMI_API int somi_moe_router_select(const float* logits, long long l_stride, int splits,
+                                    long long split_stride, const float* correction,
                                     int T, int n, int count, int keep, int top, int* chosen,
                                     float* weight, int over_chosen, int sigmoid, int group_best,
-                                    float factor, cudaStream_t stream) {
+                                    float factor, float* tail, cudaStream_t stream) {
     if (T <= 0) return 0;
-    if (n <= 0 || n > 4096 || top <= 0 || top > n || (count > 1 && (n % count || keep <= 0 || keep > count)))
+    if (n <= 0 || n > 4096 || splits < 1 || top <= 0 || top > n || (count > 1 && (n % count || keep <= 0 || keep > count)))
         return SOMI_ERR_UNSUPPORTED;
     if (count > 1 && keep < count && top > keep * (n / count)) return SOMI_ERR_UNSUPPORTED;
     if ((sigmoid && over_chosen) || group_best < 1 || group_best > 2) return SOMI_ERR_UNSUPPORTED;
     const int warps = 4;
-    const size_t smem = sizeof(float) * warps * (2 * n + (count > 1 ? count : 1));
+    const size_t smem = sizeof(float) * warps * (3 * n + (count > 1 ? count : 1));
     if (smem > 48 * 1024)
         cudaFuncSetAttribute(moe_router_select_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     launch_pdl(moe_router_select_kernel, dim3((T + warps - 1) / warps), dim3(32 * warps), smem, stream,
-               logits, l_stride, correction, n, count, keep, top, chosen, weight, T, over_chosen, sigmoid,
-               group_best, factor);
+               logits, l_stride, splits, split_stride, correction, n, count, keep, top, chosen, weight, T, over_chosen, sigmoid,
+               group_best, factor, tail);
     return launch_status();
 }
 
@@ -749,10 +768,11 @@ SOMI_API int somi_moe_combine_weighted(const void* y, int y_dtype, const int* pl
     const int vec = (H % 4 == 0 && side_stride % 4 == 0 &&
                      ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(x) |
                        reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(side)) & 15) == 0) ? 1 : 0;
-    const int threads = min(256, max(32, ((H / (vec ? 4 : 1) + 31) / 32) * 32));
-    const int blocks = min(T, 148 * 32);
+    const int per_row = (H / (vec ? 4 : 1) + 31) / 32 * 32;        // threads a row could use
+    const int threads = min(T <= 64 ? 64 : 256, max(32, per_row));
+    const dim3 blocks(min(T, 148 * 32), T <= 64 ? (per_row + threads - 1) / threads : 1);
 #define SOMI_LAUNCH_CW(TY, TX, TS)                                                                \
-    launch_pdl(moe_combine_weighted_kernel<TY, TX, TS>, dim3(blocks), dim3(threads), 0, stream,   \
+    launch_pdl(moe_combine_weighted_kernel<TY, TX, TS>, blocks, dim3(threads), 0, stream,   \
                static_cast<const TY*>(y), place, table, weight, static_cast<const TX*>(x), E, top, H, T, vec, \
                static_cast<const TS*>(side), side_splits, side_stride, side_gate, gate_stride, out)
     const bool side_f32 = side == nullptr || side_dtype == SOMI_F32;

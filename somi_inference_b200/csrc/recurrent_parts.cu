@@ -211,6 +211,96 @@ __global__ void headnorm_rotary_store_kernel(T* __restrict__ qkv, long long stri
     }
 }
 
+// The same for bfloat16 heads of 8 LANES elements: a lane holds eight neighbouring elements (one
+// 16-byte access), LANES lanes a head, so a warp takes 32 / LANES heads at once; the partner of a
+// rotated element sits in another lane of the head (needs rot / 2 a multiple of 8).
+template <int LANES>
+__global__ void headnorm_rotary_store_vec_kernel(__nv_bfloat16* __restrict__ qkv, long long stride,
+                                                 const int* __restrict__ positions,
+                                                 const double* __restrict__ inv_freq, int nq, int nkv,
+                                                 int vd, int rot, const void* __restrict__ q_w,
+                                                 const void* __restrict__ k_w, int w_dtype, float eps,
+                                                 float magnitude, int maps,
+                                                 const int* __restrict__ slot_map,
+                                                 __nv_bfloat16* __restrict__ kcache,
+                                                 __nv_bfloat16* __restrict__ vcache, int page_size) {
+    constexpr int HD = 8 * LANES;
+    extern __shared__ __align__(16) float2 cs_s[];     // [rot / 2] cosine, sine
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const int lane = threadIdx.x & 31, sub = lane % LANES;
+    __nv_bfloat16* row = qkv + static_cast<size_t>(t) * stride;
+    const double pos = static_cast<double>(positions[t]);
+    const int slot = slot_map != nullptr ? slot_map[t] : -1;
+    const size_t page = slot >= 0 ? slot / page_size : 0, off = slot >= 0 ? slot % page_size : 0;
+    const int half = rot >> 1, nv = nkv / maps;
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        const float2 cs = turn_by(pos, inv_freq[i]);
+        cs_s[i] = make_float2(cs.x * magnitude, cs.y * magnitude);
+    }
+    __syncthreads();
+    const int e0 = 8 * sub;
+    const bool turned = e0 < rot, first = e0 < half;
+    const int partner = turned ? (first ? sub + (half >> 3) : sub - (half >> 3)) : sub;
+    const int per_round = blockDim.x / LANES * gridDim.y;
+    const int mine = blockIdx.y * (blockDim.x / LANES) + threadIdx.x / LANES;
+    // (whole warps go through the rounds together: lanes past the last head shuffle, too)
+    for (int h0 = 0; h0 < nq + nkv; h0 += per_round) {
+        const int head = h0 + mine;
+        const bool live = head < nq + nkv;
+        __nv_bfloat16* x = row + static_cast<size_t>(live ? head : 0) * HD + e0;
+        const uint4 raw = *reinterpret_cast<const uint4*>(x);
+        const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&raw);
+        float v[8];
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            v[2 * j] = __low2float(h[j]);
+            v[2 * j + 1] = __high2float(h[j]);
+            ss = fmaf(v[2 * j], v[2 * j], fmaf(v[2 * j + 1], v[2 * j + 1], ss));
+        }
+        if (q_w != nullptr) {
+#pragma unroll
+            for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            const float r = 1.0f / sqrtf(ss / static_cast<float>(HD) + eps);
+            const void* w = head < nq ? q_w : k_w;
+            const F4 w0 = load4_any(w, w_dtype, e0), w1 = load4_any(w, w_dtype, e0 + 4);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                v[j] = v[j] * r * w0.v[j];
+                v[4 + j] = v[4 + j] * r * w1.v[j];
+            }
+        }
+        if (rot > 0) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const float other = __shfl_sync(0xffffffffu, v[j], partner, LANES);
+                if (turned) {
+                    const float2 cs = cs_s[(first ? e0 : e0 - half) + j];
+                    v[j] = first ? fmaf(v[j], cs.x, -(other * cs.y)) : fmaf(v[j], cs.x, other * cs.y);
+                }
+            }
+        }
+        __nv_bfloat16* dst = nullptr;
+        if (live && head < nq) dst = x;
+        else if (live && slot >= 0)
+            dst = kcache + (((page * nv + (head - nq) / maps) * page_size + off) * maps + (head - nq) % maps) * HD + e0;
+        if (dst != nullptr) {
+            store4(dst, F4{{v[0], v[1], v[2], v[3]}});
+            store4(dst + 4, F4{{v[4], v[5], v[6], v[7]}});
+        }
+    }
+    if (slot >= 0 && blockIdx.y == gridDim.y - 1) {
+        const __nv_bfloat16* vrow = row + static_cast<size_t>(nq + nkv) * HD;
+        for (int c = threadIdx.x; c < nv * (vd >> 3); c += blockDim.x) {
+            const int g = c / (vd >> 3), e = (c - g * (vd >> 3)) * 8;
+            *reinterpret_cast<uint4*>(vcache + ((page * nv + g) * page_size + off) * vd + e) =
+                *reinterpret_cast<const uint4*>(vrow + static_cast<size_t>(g) * vd + e);
+        }
+    }
+}
+
 // ------------------------------------------------------- matrix-state recurrence
 // Per request r and head h a state S [dk, dv] float32 in the request's slot (stored column by
 // column, [dv][dk]); per token, in order:
@@ -814,6 +904,29 @@ SOMI_API int somi_headnorm_rotary_store(void* qkv, int dtype, long long stride, 
     if (hd <= 0 || hd > 1024 || vd <= 0 || rot < 0 || rot > hd || (rot & 1) || nq <= 0 || nkv <= 0 ||
         maps <= 0 || nkv % maps)
         return SOMI_ERR_UNSUPPORTED;
+    auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    if (dtype == SOMI_BF16 && (hd == 16 || hd == 32 || hd == 64 || hd == 128 || hd == 256) && vd % 8 == 0 &&
+        rot % 16 == 0 && stride % 8 == 0 && aligned(qkv) && aligned(kcache) && aligned(vcache) && aligned(q_w) &&
+        aligned(k_w)) {
+        const int lanes = hd / 8;
+        const int threads = min(256, ((nq + nkv) * lanes + 31) / 32 * 32);
+        const dim3 vgrid(T, T <= 256 ? ((nq + nkv) * lanes + threads - 1) / threads : 1);
+        const size_t vsmem = sizeof(float2) * (rot >> 1);
+#define SOMI_LAUNCH_HRV(L)                                                                         \
+    launch_pdl(headnorm_rotary_store_vec_kernel<L>, vgrid, dim3(threads), vsmem, stream,           \
+               static_cast<__nv_bfloat16*>(qkv), stride, positions, inv_freq, nq, nkv, vd, rot,    \
+               q_w, k_w, w_dtype, eps, magnitude, maps, slot_map, static_cast<__nv_bfloat16*>(kcache), \
+               static_cast<__nv_bfloat16*>(vcache), page_size)
+        switch (lanes) {
+            case 2: SOMI_LAUNCH_HRV(2); break;
+            case 4: SOMI_LAUNCH_HRV(4); break;
+            case 8: SOMI_LAUNCH_HRV(8); break;
+            case 16: SOMI_LAUNCH_HRV(16); break;
+            default: SOMI_LAUNCH_HRV(32); break;
+        }
+#undef SOMI_LAUNCH_HRV
+        return launch_status();
+    }
     const int warps = min(8, nq + nkv);
     const dim3 grid(T, T <= 256 ? (nq + nkv + 7) / 8 : 1);
     const size_t smem = sizeof(float) * warps * hd + sizeof(float2) * (rot >> 1);

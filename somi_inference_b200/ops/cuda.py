@@ -1620,7 +1620,7 @@ class CudaOps:
 
     def moe_router_select(self, logits, correction, count: int, keep: int, top: int,
                           over_chosen: bool = False, sigmoid: bool = False, group_best: int = 1,
-                          outputs: int | None = None, factor: float = 1.0):
+                          outputs: int | None = None, factor: float = 1.0, tail: bool = False):
         """logits float32 [T, n] -> (chosen int32 [T, top], weight float32 [T, top]): softmax over
         the n outputs; the choice is made on softmax + correction (None: the softmax) among the
         members of the `keep` best of `count` equal groups of neighbours (a group's score is its
@@ -1628,23 +1628,30 @@ class CudaOps:
         `over_chosen`: the `top` largest logits are chosen (no correction, no groups) and the
         weights are the softmax over the chosen logits only.  `sigmoid`: sigmoids of the logits take the
         softmax's place; `group_best` 2: a group's score is the sum of its two best members'.  `outputs`: only
-        the first so many columns of `logits` are router outputs; `factor` multiplies all weights."""
+        the first so many columns of `logits` are router outputs; `factor` multiplies all weights.  The
+        logits may be float32 [splits, T, n] partial sums, added in order.  `tail`: a third result,
+        float32 [T], is the (summed) column behind the router outputs."""
         _check(logits, correction)
         assert logits.dtype == torch.float32 and (correction is None or correction.dtype == torch.float32)
-        T, n = logits.shape[0], outputs if outputs is not None else logits.shape[1]
+        T, n = logits.shape[-2], outputs if outputs is not None else logits.shape[-1]
+        splits = logits.shape[0] if logits.dim() == 3 else 1
+        assert n + (1 if tail else 0) <= logits.shape[-1]
+        behind = torch.empty(T, dtype=torch.float32, device=logits.device) if tail else None
         chosen = torch.empty((T, top), dtype=torch.int32, device=logits.device)
         weight = torch.empty((T, top), dtype=torch.float32, device=logits.device)
-        rc = self.lib.somi_moe_router_select(_ptr(logits), ctypes.c_longlong(logits.stride(0)),
+        rc = self.lib.somi_moe_router_select(_ptr(logits), ctypes.c_longlong(logits.shape[-1]),
+                                             ctypes.c_int(splits),
+                                             ctypes.c_longlong(T * logits.shape[-1]),
                                              _ptr(correction), ctypes.c_int(T), ctypes.c_int(n),
                                              ctypes.c_int(count), ctypes.c_int(keep), ctypes.c_int(top),
                                              _ptr(chosen), _ptr(weight),
                                              ctypes.c_int(1 if over_chosen else 0),
                                              ctypes.c_int(1 if sigmoid else 0), ctypes.c_int(group_best),
-                                             ctypes.c_float(factor), self._stream())
+                                             ctypes.c_float(factor), _ptr(behind), self._stream())
         self._done(rc, "moe_router_select")
         if trace.active():
-            trace.note("moe_router_select", T * (n * 4 + top * 8))
-        return chosen, weight
+            trace.note("moe_router_select", T * (splits * n * 4 + top * 8))
+        return (chosen, weight, behind) if tail else (chosen, weight)
 
     def moe_combine_weighted(self, y, place, table, weight, x, num_experts: int, side=None,
                              side_gate=None) -> torch.Tensor:

@@ -209,7 +209,7 @@ class RoutedMoE:
             self.gated = None
         self.w_down = torch.stack([tensors[n["down"][e]] for e in E]).contiguous()
 
-    def _side(self, x: torch.Tensor, logits: torch.Tensor) -> dict:
+    def _side(self, x: torch.Tensor, gate_logits: torch.Tensor | None) -> dict:
         """The shared expert's result (few tokens: split-K partial sums, added up by the weighted sum)
         and its gate's logits, as the weighted sum takes them."""
         if self.shared is None:
@@ -220,16 +220,20 @@ class RoutedMoE:
             act = self.ctx.ops.clamped_gate_up(gate_up(x), *form)
         side = down.partial_sums(act)
         return {"side": down(act) if side is None else side,
-                "side_gate": logits[:, self.outputs] if self.token_gate else None}
+                "side_gate": gate_logits}
 
     def forward(self, x: torch.Tensor, batch) -> torch.Tensor:
         ops, top, E = self.ctx.ops, self.top, self.experts
-        logits = self.router.to_float32(x)
-        chosen, weight = ops.moe_router_select(logits, self.correction, self.group_count,
+        # few tokens: split-K partial sums of the one product, added up where the choice is made
+        logits = self.router.partial_sums(x)
+        if logits is None:
+            logits = self.router.to_float32(x)
+        chosen, weight, *gate = ops.moe_router_select(logits, self.correction, self.group_count,
                                                self.group_keep, top, over_chosen=self.over_chosen,
                                                sigmoid=self.sigmoid, group_best=self.group_best,
-                                               outputs=self.outputs, factor=self.factor)
-        side = self._side(x, logits)
+                                               outputs=self.outputs, factor=self.factor,
+                                               tail=self.token_gate)
+        side = self._side(x, gate[0] if gate else None)
         n_entries = x.shape[0] * top
         if ops.moe_gemv_supported(n_entries, x.shape[1], x.dtype) and self.w_down.shape[2] % 8 == 0:
             act = ops.moe_gemv(x, self.w_gate_up, None, chosen, per_token=True, gated=self.gated,

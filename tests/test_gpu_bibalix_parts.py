@@ -90,14 +90,16 @@ def test_layer_norm_with_a_bias(ops, dtype, width, tokens):
 @pytest.mark.parametrize("case", [
     # (heads, kv heads, key width, value width, rotated, normed, scaling factor, columns behind)
     (4, 2, 12, 28, 8, True, None, 0), (1, 1, 5, 3, 4, True, 8.0, 3), (3, 1, 10, 8, 10, True, None, 1),
-    (6, 2, 64, 128, 32, True, None, 8), (2, 2, 32, 64, 0, True, None, 0), (8, 1, 16, 32, 16, False, 2.0, 0)])
+    (6, 2, 64, 128, 32, True, None, 8), (2, 2, 32, 64, 0, True, None, 0), (8, 1, 16, 32, 16, False, 2.0, 0),
+    (30, 5, 64, 128, 48, True, 4.0, 40), (1, 1, 128, 256, 128, True, None, 8), (2, 1, 256, 8, 16, True, 8.0, 8),
+    (9, 3, 32, 24, 16, False, None, 0)])
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_two_queries_and_two_keys_a_head(ops, dtype, case):
     H, G, d, dv, rot, normed, factor, pad = case
     g = torch.Generator().manual_seed(d + dv)
     steps = Steps(ops, 2, paged=PagedKVNeeds(G, 2 * d, None, dv if dv != 2 * d else None), dtype=dtype, page_size=4)
     steps.step({"a": 30})
-    batch, where = steps.step({"a": 5, "b": 7})
+    batch, where = steps.step({"a": 5, "b": 7} if H < 30 else {"a": 300, "b": 1})
     wide = torch.randn((batch.num_tokens, 2 * (H + G) * d + G * dv + pad), generator=g).to(dtype).cuda()
     qkv = wide.clone()
     qw = (1 + 0.3 * torch.randn(d, generator=g)).to(dtype).cuda() if normed else None
@@ -317,6 +319,16 @@ def test_router_softmax_over_all_times_a_factor(ops, n, top, factor, behind):
     idx, wt = plain.choose_experts(z, {"top": top, "scale": factor})
     assert torch.equal(chosen.cpu().long(), idx)
     assert (weight.double().cpu() - wt).abs().max().item() < 1e-6
+    # the same from partial sums, and the column behind the outputs summed beside it
+    parts = torch.randn((5, *logits.shape), generator=g).cuda()
+    parts[-1] += logits - parts.sum(0)
+    again, w2, *behind_sum = ops.moe_router_select(parts, None, 1, 1, top, outputs=n, factor=factor, tail=behind > 0)
+    z = parts.double().sum(0).cpu()
+    clear = plain.choice_margin(z[:, :n], {"top": top}) > 1e-4
+    assert torch.equal(again.cpu().long()[clear], idx[clear]) and clear.sum() > 50
+    assert (w2.double().cpu() - wt)[clear].abs().max().item() < 1e-5
+    if behind:
+        assert (behind_sum[0].double().cpu() - z[:, n]).abs().max().item() < 1e-4
 
 
 @pytest.mark.parametrize("tokens", [1, 5, 16, 40, 130])
