@@ -457,65 +457,65 @@ paged_prefill_pp_kernel(const __grid_constant__ CUtensorMap q_map,
                     }
                 }
             } else {
-            if (!ok) failed_s = 1;
-            // a sink: one more score in the denominator, without a value
-            if (sinks != nullptr) l += fast_exp2(sinks[head] * 1.4426950408889634f - m);
-            const float inv = 1.0f / l;
-            const int r = x * kPpBM + row;
-            __nv_bfloat16* dst = out + static_cast<size_t>(row0 + r) * nq * HD + head * HD;
-            auto store8 = [](__nv_bfloat16* p, const float* y) {
-                uint4 w;
-                w.x = pack_bf16(y[0], y[1]);
-                w.y = pack_bf16(y[2], y[3]);
-                w.z = pack_bf16(y[4], y[5]);
-                w.w = pack_bf16(y[6], y[7]);
-                *reinterpret_cast<uint4*>(p) = w;
-            };
-            if (turn == nullptr) {
+                if (!ok) failed_s = 1;
+                // a sink: one more score in the denominator, without a value
+                if (sinks != nullptr) l += fast_exp2(sinks[head] * 1.4426950408889634f - m);
+                const float inv = 1.0f / l;
+                const int r = x * kPpBM + row;
+                __nv_bfloat16* dst = out + static_cast<size_t>(row0 + r) * nq * HD + head * HD;
+                auto store8 = [](__nv_bfloat16* p, const float* y) {
+                    uint4 w;
+                    w.x = pack_bf16(y[0], y[1]);
+                    w.y = pack_bf16(y[2], y[3]);
+                    w.z = pack_bf16(y[4], y[5]);
+                    w.w = pack_bf16(y[6], y[7]);
+                    *reinterpret_cast<uint4*>(p) = w;
+                };
+                if (turn == nullptr) {
 #pragma unroll
-                for (int c = 0; c < HD / 32; ++c) {
-                    uint32_t v[32];
-                    t5::ld32_nowait(o_addr + c * 32, v);
-                    t5::wait_ld();
-                    if (r < rows) {
+                    for (int c = 0; c < HD / 32; ++c) {
+                        uint32_t v[32];
+                        t5::ld32_nowait(o_addr + c * 32, v);
+                        t5::wait_ld();
+                        if (r < rows) {
 #pragma unroll
-                        for (int d = 0; d < 32; d += 8) {
-                            float y[8];
+                            for (int d = 0; d < 32; d += 8) {
+                                float y[8];
 #pragma unroll
-                            for (int j = 0; j < 8; ++j) y[j] = __uint_as_float(v[d + j]) * inv;
-                            store8(dst + c * 32 + d, y);
-                        }
-                    }
-                }
-            } else {
-                // the pairs (d, d + HD / 2) are turned back by the row's angles before they are rounded
-#pragma unroll
-                for (int c = 0; c < HD / 64; ++c) {
-                    uint32_t v[32], u[32];
-                    t5::ld32_nowait(o_addr + c * 32, v);
-                    t5::ld32_nowait(o_addr + HD / 2 + c * 32, u);
-                    t5::wait_ld();
-                    if (r < rows) {
-                        const float4* tr = reinterpret_cast<const float4*>(turn + static_cast<size_t>(row0 + r) * (HD / 2) + c * 32);
-#pragma unroll
-                        for (int d = 0; d < 32; d += 8) {
-                            float y0[8], y1[8];
-#pragma unroll
-                            for (int j = 0; j < 8; j += 2) {
-                                const float4 cs = tr[(d + j) / 2];          // two pairs' cosine, sine
-                                const float p0 = __uint_as_float(v[d + j]) * inv, q0 = __uint_as_float(u[d + j]) * inv;
-                                const float p1 = __uint_as_float(v[d + j + 1]) * inv, q1 = __uint_as_float(u[d + j + 1]) * inv;
-                                y0[j] = fmaf(p0, cs.x, q0 * cs.y);
-                                y1[j] = fmaf(q0, cs.x, -(p0 * cs.y));
-                                y0[j + 1] = fmaf(p1, cs.z, q1 * cs.w);
-                                y1[j + 1] = fmaf(q1, cs.z, -(p1 * cs.w));
+                                for (int j = 0; j < 8; ++j) y[j] = __uint_as_float(v[d + j]) * inv;
+                                store8(dst + c * 32 + d, y);
                             }
-                            store8(dst + c * 32 + d, y0);
-                            store8(dst + HD / 2 + c * 32 + d, y1);
+                        }
+                    }
+                } else {
+                    // the pairs (d, d + HD / 2) are turned back by the row's angles before they are rounded
+#pragma unroll
+                    for (int c = 0; c < HD / 64; ++c) {
+                        uint32_t v[32], u[32];
+                        t5::ld32_nowait(o_addr + c * 32, v);
+                        t5::ld32_nowait(o_addr + HD / 2 + c * 32, u);
+                        t5::wait_ld();
+                        if (r < rows) {
+                            const float4* tr = reinterpret_cast<const float4*>(turn + static_cast<size_t>(row0 + r) * (HD / 2) + c * 32);
+#pragma unroll
+                            for (int d = 0; d < 32; d += 8) {
+                                float y0[8], y1[8];
+#pragma unroll
+                                for (int j = 0; j < 8; j += 2) {
+                                    const float4 cs = tr[(d + j) / 2];          // two pairs' cosine, sine
+                                    const float p0 = __uint_as_float(v[d + j]) * inv, q0 = __uint_as_float(u[d + j]) * inv;
+                                    const float p1 = __uint_as_float(v[d + j + 1]) * inv, q1 = __uint_as_float(u[d + j + 1]) * inv;
+                                    y0[j] = fmaf(p0, cs.x, q0 * cs.y);
+                                    y1[j] = fmaf(q0, cs.x, -(p0 * cs.y));
+                                    y0[j + 1] = fmaf(p1, cs.z, q1 * cs.w);
+                                    y1[j + 1] = fmaf(q1, cs.z, -(p1 * cs.w));
+                                }
+                                store8(dst + c * 32 + d, y0);
+                                store8(dst + HD / 2 + c * 32 + d, y1);
+                            }
                         }
                     }
                 }
-            }
             }
         }
     }
